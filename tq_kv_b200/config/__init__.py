@@ -2,6 +2,9 @@
 from .furesun import ARCHITECTURE as FURESUN_ARCHITECTURE
 from .furesun import MODEL_TYPE as FURESUN_MODEL_TYPE
 from .furesun import FuresunConfig, build_furesun_spec
+from .gokapel import ARCHITECTURE as GOKAPEL_ARCHITECTURE
+from .gokapel import MODEL_TYPE as GOKAPEL_MODEL_TYPE
+from .gokapel import GokapelConfig, build_gokapel_spec
 from .model_spec import ConfigError, LayerSpec, ModelSpec, PartSpec, ScheduleEntry
 from .pavisun import ARCHITECTURE as PAVISUN_ARCHITECTURE
 from .pavisun import MODEL_TYPE as PAVISUN_MODEL_TYPE
@@ -34,7 +37,11 @@ register_architecture(
 register_architecture(
     Architecture(FURESUN_ARCHITECTURE, FURESUN_MODEL_TYPE, FuresunConfig, build_furesun_spec), replace=True)
 
+register_architecture(
+    Architecture(GOKAPEL_ARCHITECTURE, GOKAPEL_MODEL_TYPE, GokapelConfig, build_gokapel_spec), replace=True)
+
 __all__ = [
+    "GokapelConfig", "build_gokapel_spec",
     "FuresunConfig", "build_furesun_spec",
     "PavisunConfig", "build_pavisun_spec",
     "RirudraConfig", "build_rirudra_spec",

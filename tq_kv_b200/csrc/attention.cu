@@ -12,9 +12,11 @@
 // Options beyond the reference (AttnOptions; all off by default): value rows
 // of another width than the keys; a cap on the scores, s <- cap * tanh(s / cap);
 // a bias that grows with the distance, s <- s - slope[h] * (p - j); and first
-// tokens that stay visible behind the window (keys j < keep_first); a sink in
-// the softmax: one more key of score 0 that has no value, i.e. one added to the
-// softmax's denominator (in the merge step where the keys are split).
+// tokens that stay visible behind the window (keys j < keep_first); instead of a
+// window, chunks: the query at position p sees the keys of its own chunk of
+// `chunk` positions, p - p % chunk .. p; a sink in the softmax: one more key of
+// head h with the score sinks[h] that has no value, i.e. exp(sinks[h]) added to
+// the softmax's denominator (in the merge step where the keys are split).
 #include "common.cuh"
 
 #define ATT_MAX_PAIRS 8   // head_dim <= 512: each lane owns up to 8 pairs of dims
@@ -37,7 +39,8 @@ struct AttnOptions {
     float softcap;          // > 0: scores become softcap * tanh(score / softcap)
     const float* slopes;    // [nh] or null: score -= slopes[h] * (query position - key position)
     int keep_first;         // with a window: keys below this position stay visible
-    int sink;               // != 0: the softmax's denominator counts one more key of score 0 (it has no value)
+    const float* sinks;     // [nh] or null: the softmax's denominator counts one more key of score sinks[h] (no value)
+    int chunk;              // > 0 (then no window): keys of the query's own chunk of this many positions only
 };
 
 template <typename TC>
@@ -72,7 +75,8 @@ __global__ void attention_kernel(const TC* __restrict__ q, KVSource src, const i
     const int pos = tok_pos[t];
     const int b = tok_seq[t];
     const int tok0 = src.k_packed ? cu_seqlens[b] - start_pos[b] : 0;
-    const int lo_all = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo_all = opt.chunk > 0 ? pos - pos % opt.chunk
+                                     : ((window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0);
     // The visible keys, counted 0 .. n_keys-1: first the kept first tokens that the window has left behind
     // (n_keep of them, positions 0 .. n_keep-1), then the window's keys lo_all .. pos.
     const int n_keep = opt.keep_first < lo_all ? opt.keep_first : lo_all;
@@ -143,10 +147,11 @@ __global__ void attention_kernel(const TC* __restrict__ q, KVSource src, const i
         }
 
         if (n_splits == 1) {
-            if (opt.sink) {                                  // the sink's exp(0 - m), with the maximum moved up to 0
-                const float m_new = fmaxf(m, 0.f);
+            if (opt.sinks) {                                 // the sink's exp(sink - m), the maximum moved up to it
+                const float sink = opt.sinks[h];
+                const float m_new = fmaxf(m, sink);
                 const float corr = expf(m - m_new);
-                l = l * corr + expf(-m_new);
+                l = l * corr + expf(sink - m_new);
 #pragma unroll
                 for (int i = 0; i < 2 * ATT_MAX_PAIRS; ++i) acc[i] *= corr;
             }
@@ -175,7 +180,8 @@ __global__ void attention_kernel(const TC* __restrict__ q, KVSource src, const i
 // scheduling.  An empty split has m = -inf and l = 0 and contributes nothing.
 template <typename TC>
 __global__ void attention_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                       TC* __restrict__ out, int nh, int hd, int n_splits, int sink) {
+                                       TC* __restrict__ out, int nh, int hd, int n_splits,
+                                       const float* __restrict__ sinks) {
     const size_t r0 = ((size_t)blockIdx.x * nh + blockIdx.y) * n_splits;
     const int lane = threadIdx.x & 31;
     pdl_wait();
@@ -184,14 +190,15 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_acc, const
     float m = -INFINITY;
     for (int s = lane; s < n_splits; s += 32) m = fmaxf(m, part_ml[2 * (r0 + s)]);
     m = warp_max(m);
-    if (sink) m = fmaxf(m, 0.f);                    // the sink is one more split: maximum 0, sum 1, no values
+    const float sink = sinks ? sinks[blockIdx.y] : 0.f;
+    if (sinks) m = fmaxf(m, sink);                  // the sink is one more split: maximum `sink`, sum 1, no values
     float l = 0.f;
     for (int s = lane; s < n_splits; s += 32) {
         const float ms = part_ml[2 * (r0 + s)];
         if (ms > -INFINITY) l += part_ml[2 * (r0 + s) + 1] * expf(ms - m);
     }
     l = warp_sum(l);
-    if (sink) l += expf(-m);
+    if (sinks) l += expf(sink - m);
     TC* o = out + ((size_t)blockIdx.x * nh + blockIdx.y) * hd;
     for (int d = threadIdx.x; d < hd; d += blockDim.x) {
         float a = 0.f;
@@ -213,7 +220,7 @@ TQ_API int tq_attention_ext(const void* q, int dtype, const void* k_packed, cons
                             int page_tokens, const int* tok_pos, const int* tok_seq, const int* cu_seqlens,
                             const int* start_pos, int window, float scale, void* out, float* part_acc, float* part_ml,
                             int n_tokens, int nh, int nkv, int hd, int vd, float softcap, const float* slopes,
-                            int keep_first, int sink, int n_splits, cudaStream_t stream) {
+                            int keep_first, const float* sinks, int chunk, int n_splits, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (hd <= 0 || hd > 64 * ATT_MAX_PAIRS || hd % 8 || nkv <= 0 || nh % nkv) return (int)cudaErrorInvalidValue;
     if (vd <= 0 || vd > 64 * ATT_MAX_PAIRS || vd % 8 || keep_first < 0) return (int)cudaErrorInvalidValue;
@@ -222,7 +229,8 @@ TQ_API int tq_attention_ext(const void* q, int dtype, const void* k_packed, cons
     if (!k_packed && (!k_pages || !block_table || page_tokens <= 0)) return (int)cudaErrorInvalidValue;
     if (nkv > 65535 || n_splits > 65535) return (int)cudaErrorInvalidValue;
     KVSource src{k_packed, v_packed, k_pages, v_pages, block_table, table_width, ring_pages, page_tokens};
-    AttnOptions opt{vd, softcap, slopes, window > 0 ? keep_first : 0, sink};
+    if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
+    AttnOptions opt{vd, softcap, slopes, window > 0 ? keep_first : 0, sinks, chunk};
     const int n_rep = nh / nkv;
     const int n_warps = n_rep < 8 ? n_rep : 8;
     const dim3 grid(n_tokens, nkv, n_splits);
@@ -241,9 +249,9 @@ TQ_API int tq_attention_ext(const void* q, int dtype, const void* k_packed, cons
     if (st || n_splits == 1) return st;
     const dim3 mgrid(n_tokens, nh);
     if (dtype == TQ_F32)
-        attention_merge_kernel<float><<<mgrid, 128, 0, stream>>>(part_acc, part_ml, (float*)out, nh, vd, n_splits, sink);
+        attention_merge_kernel<float><<<mgrid, 128, 0, stream>>>(part_acc, part_ml, (float*)out, nh, vd, n_splits, sinks);
     else
-        attention_merge_kernel<bf16><<<mgrid, 128, 0, stream>>>(part_acc, part_ml, (bf16*)out, nh, vd, n_splits, sink);
+        attention_merge_kernel<bf16><<<mgrid, 128, 0, stream>>>(part_acc, part_ml, (bf16*)out, nh, vd, n_splits, sinks);
     return tq_launch_status();
 }
 
@@ -255,20 +263,20 @@ TQ_API int tq_attention(const void* q, int dtype, const void* k_packed, const vo
     if (hd % 16) return (int)cudaErrorInvalidValue;
     return tq_attention_ext(q, dtype, k_packed, v_packed, k_pages, v_pages, block_table, table_width, ring_pages,
                             page_tokens, tok_pos, tok_seq, cu_seqlens, start_pos, window, scale, out, part_acc,
-                            part_ml, n_tokens, nh, nkv, hd, hd, 0.f, nullptr, 0, 0, n_splits, stream);
+                            part_ml, n_tokens, nh, nkv, hd, hd, 0.f, nullptr, 0, nullptr, 0, n_splits, stream);
 }
 
 // The merge step alone, for kernels that write (unnormalised output, max, sum) per split themselves.
 TQ_API int tq_attention_merge(const float* part_acc, const float* part_ml, void* out, int dtype, int n_tokens, int nh,
-                              int hd, int n_splits, int sink, cudaStream_t stream) {
+                              int hd, int n_splits, const float* sinks, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_splits < 1 || !part_acc || !part_ml) return (int)cudaErrorInvalidValue;
     const dim3 mgrid(n_tokens, nh);
     if (dtype == TQ_F32)
         return tq_launch_pdl(TQ_PDL_MERGE, attention_merge_kernel<float>, mgrid, dim3(128), 0, stream, part_acc, part_ml,
-                             (float*)out, nh, hd, n_splits, sink);
+                             (float*)out, nh, hd, n_splits, sinks);
     if (dtype == TQ_BF16)
         return tq_launch_pdl(TQ_PDL_MERGE, attention_merge_kernel<bf16>, mgrid, dim3(128), 0, stream, part_acc, part_ml,
-                             (bf16*)out, nh, hd, n_splits, sink);
+                             (bf16*)out, nh, hd, n_splits, sinks);
     return (int)cudaErrorInvalidValue;
 }

@@ -111,6 +111,9 @@ __device__ __forceinline__ float block_max(float v, float* red) {
 // and division (a couple of float32 ulp: for results that are rounded to bfloat16).
 #define TQ_ACT_SILU 1
 #define TQ_ACT_GELU_TANH 2
+// Not of a gated product: the square of relu on a plain product's result (after its bias).
+#define TQ_ACT_SQUARE_RELU 3
+__device__ __forceinline__ float square_relu(float z) { const float p = fmaxf(z, 0.f); return p * p; }
 __device__ __forceinline__ float gated_act(float z, int act) {
     if (act == TQ_ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     return z / (1.f + expf(-z));

@@ -84,8 +84,9 @@ __device__ __forceinline__ void dg_ld32(uint32_t taddr, float* v) {
 // summed on the way, each block over its share of K, and the shares meet with the partial products in the
 // cluster's exchange, where every output is scaled by 1 / sqrt(mean(h^2) + eps) of its batch row.  So the norm
 // needs no kernel and no trip through memory of its own.
-// The gate's activation of a gated product (TQ_ACT_*): the exported functions set it from their `swiglu` argument
-// (1 or 2; 0: not gated) right before they launch, on the launching thread.
+// The gate's activation of a gated product (TQ_ACT_*), or TQ_ACT_SQUARE_RELU on a plain one with a bfloat16 result
+// (its K is never cut into independent shares): the exported functions set it from their `swiglu` argument (1 or 2:
+// gated; 3: plain, squared relu; 0: plain) right before they launch, on the launching thread.
 static thread_local int dg_gate_act = TQ_ACT_SILU;
 #define DG_NORM_ROWS 16
 #define DG_HRING 4
@@ -408,6 +409,8 @@ decode_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
                 if (bias) { v += bias[col]; if (SWIGLU) w += bias[col + N]; }
                 if (SWIGLU)            // (a bfloat16 result keeps 8 bits: the fast exponential and division do)
                     v = (sizeof(TO) == 2 ? gated_act_fast(v, act) : gated_act(v, act)) * w;
+                else if (act == TQ_ACT_SQUARE_RELU)
+                    v = square_relu(v);
                 TO* y = Y + (size_t)m * ldy + col;
                 if (accumulate) v += to_f32<TO>(*y);
                 *y = from_f32<TO>(v);
@@ -557,8 +560,10 @@ TQ_API int tq_decode_gemm_tc(const void* X, const void* W, const float* bias, vo
     if ((reinterpret_cast<uintptr_t>(X) & 15) || (reinterpret_cast<uintptr_t>(W) & 15))
         return (int)cudaErrorInvalidValue;
     if (accumulate && y_dtype != TQ_F32) return (int)cudaErrorInvalidValue;
-    if (swiglu != 0 && swiglu != TQ_ACT_SILU && swiglu != TQ_ACT_GELU_TANH) return (int)cudaErrorInvalidValue;
+    if (swiglu < 0 || swiglu > TQ_ACT_SQUARE_RELU || (swiglu == TQ_ACT_SQUARE_RELU && y_dtype != TQ_BF16))
+        return (int)cudaErrorInvalidValue;
     dg_gate_act = swiglu ? swiglu : TQ_ACT_SILU;
+    if (swiglu == TQ_ACT_SQUARE_RELU) swiglu = 0;
     const int mp = M <= 32 ? 32 : 64;
     CUtensorMap mw, mx;
     int st = dg_make_map(&mw, W, swiglu ? 2ull * N : (uint64_t)N, (uint64_t)K, (uint64_t)ldw,

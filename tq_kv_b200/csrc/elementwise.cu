@@ -741,3 +741,32 @@ TQ_API int tq_scale_inplace(float* x, size_t total, float s, cudaStream_t stream
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, scale_inplace_kernel, dim3((int)blocks), dim3(threads), 0, stream, x, total,
                          s);
 }
+
+// ---------------------------------------------------------------------------
+// out = (max(x, 0))^2, row by row (x float32 [rows, ldx], out [rows, n] contiguous): the activation behind products
+// whose kernel has no such epilogue (the float32 path's tiled product, the library's).
+// ---------------------------------------------------------------------------
+template <typename TO>
+__global__ void square_relu_kernel(const float* x, int ldx, TO* out, int n, size_t total) {
+    pdl_wait();
+    pdl_launch();
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = idx / n;
+        out[idx] = from_f32<TO>(square_relu(x[t * ldx + (idx - t * n)]));
+    }
+}
+
+TQ_API int tq_square_relu(const float* x, int ldx, void* out, int out_dtype, int n_rows, int n, cudaStream_t stream) {
+    const size_t total = (size_t)n_rows * n;
+    if (total == 0) return 0;
+    if (!x || !out || ldx < n) return (int)cudaErrorInvalidValue;
+    size_t blocks = (total + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    if (out_dtype == TQ_F32)
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, square_relu_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, x,
+                             ldx, (float*)out, n, total);
+    if (out_dtype == TQ_BF16)
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, square_relu_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, x,
+                             ldx, (bf16*)out, n, total);
+    return (int)cudaErrorInvalidValue;
+}

@@ -50,7 +50,8 @@ __device__ __forceinline__ uint32_t fd_pack(float a, float b) {
 // kernel that adds the splits does that.
 // FD_SOFTMAX_EXT: the softmax with options (FdOptions): score * scale, capped by cap * tanh(. / cap), minus
 // slopes[h] * (i - j); behind a window the first keep_first keys stay in view.  The visible keys are counted
-// 0 .. n_keys-1: first the kept ones that the window has left behind, then the window's.
+// 0 .. n_keys-1: first the kept ones that the window has left behind, then the window's.  With `chunk` (and no
+// window) the query at position p sees the keys p - p % chunk .. p.
 #define FD_SOFTMAX 0
 #define FD_SIGMOID 1
 #define FD_SOFTMAX_EXT 2
@@ -60,7 +61,8 @@ struct FdOptions {
     float softcap;          // > 0: scores become softcap * tanh(score / softcap)
     const float* slopes;    // [nh] or null
     int keep_first;         // with a window: keys below this position stay visible
-    int sink;               // != 0: one added to the softmax's denominator (a key of score 0 without a value)
+    const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
+    int chunk;              // > 0: keys of the query's own chunk only
 };
 
 // cap * tanh(x / cap) with 2^x and the reciprocal of the special-function unit (a few ulp; tanh.approx is not enough)
@@ -81,7 +83,7 @@ flash_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
                     bf16* __restrict__ out, float* __restrict__ part_acc, float* __restrict__ part_ml, int nh, int nkv,
                     int n_splits, const float* __restrict__ bias = nullptr, int n_dist = 0,
                     const float* __restrict__ gate = nullptr, int ldg = 0, int kv_div = 1,
-                    FdOptions opt = FdOptions{0.f, 0.f, nullptr, 0}) {
+                    FdOptions opt = FdOptions{0.f, 0.f, nullptr, 0, nullptr, 0}) {
     // kv_div > 1: more than 16 q heads share a key/value head; they are cut into kv_div groups, each a block row of
     // its own (nkv counts those groups), and group g reads the cache rows of head g / kv_div
     constexpr int ROW = HD * 2 + 16;                       // bytes per key row in shared memory (padded)
@@ -97,7 +99,8 @@ flash_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
     const int n_rep = nh / nkv;
     const int pos = tok_pos[t];
     const int b = tok_seq[t];
-    const int lo_all = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    int lo_all = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    if (WEIGHTS == FD_SOFTMAX_EXT && opt.chunk > 0) lo_all = pos - pos % opt.chunk;
     // the visible keys, counted 0 .. n_keys-1 (count c is position key_pos(c)): the kept first tokens that the
     // window has left behind (none unless FD_SOFTMAX_EXT), then the window's keys lo_all .. pos
     const int n_keep = (WEIGHTS == FD_SOFTMAX_EXT && opt.keep_first < lo_all) ? opt.keep_first
@@ -352,9 +355,10 @@ flash_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
         }
         const int h = g * n_rep + r;
         if (n_splits == 1) {
-            if (WEIGHTS == FD_SOFTMAX_EXT && opt.sink) {      // (with splits the merge step adds the sink)
-                const float m2 = fmaxf(m, 0.f), f = exp2f(m - m2);
-                l = l * f + exp2f(-m2);
+            if (WEIGHTS == FD_SOFTMAX_EXT && opt.sinks) {     // (with splits the merge step adds the sink)
+                const float sink = opt.sinks[h] * 1.4426950408889634f;
+                const float m2 = fmaxf(m, sink), f = exp2f(m - m2);
+                l = l * f + exp2f(sink - m2);
                 a *= f;
             }
             out[((size_t)t * nh + h) * HD + d] = __float2bfloat16_rn(a / l);
@@ -375,7 +379,7 @@ static int launch_flash_decode(const bf16* q, const bf16* kp, const bf16* vp, co
                                bf16* out, float* part_acc, float* part_ml, int n_tokens, int nh, int nkv, int n_splits,
                                int pdl_family, cudaStream_t stream, const float* bias = nullptr, int n_dist = 0,
                                const float* gate = nullptr, int ldg = 0, int kv_div = 1,
-                               FdOptions opt = FdOptions{0.f, 0.f, nullptr, 0}) {
+                               FdOptions opt = FdOptions{0.f, 0.f, nullptr, 0, nullptr, 0}) {
     constexpr int ROW = HD * 2 + 16;
     constexpr int FD_CHUNK = (HD <= 64 || !VT) ? 32 : 16;
     constexpr size_t stage_bytes = (size_t)FD_WARPS * FD_STAGES * (VT ? 2 : 1) * FD_CHUNK * ROW;
@@ -479,7 +483,8 @@ TQ_API int tq_sigmoid_flash_decode(const void* q, const void* k_pages, const voi
 // cache that keeps all keys (no ring).  Returns cudaErrorNotSupported (801) for shapes outside this kernel's reach.
 TQ_API int tq_flash_decode_ext(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                int table_width, int ring_pages, int page_tokens, const int* tok_pos, const int* tok_seq,
-                               int window, float scale, float softcap, const float* slopes, int keep_first, int sink,
+                               int window, float scale, float softcap, const float* slopes, int keep_first,
+                               const float* sinks, int chunk,
                                void* out, float* part_acc, float* part_ml, int n_tokens, int nh, int nkv, int hd,
                                int n_splits, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
@@ -491,7 +496,8 @@ TQ_API int tq_flash_decode_ext(const void* q, const void* k_pages, const void* v
     nkv *= kv_div;
     if (nkv > 65535 || n_splits > 65535) return (int)cudaErrorNotSupported;
     if (n_splits < 1 || (n_splits > 1 && (!part_acc || !part_ml))) return (int)cudaErrorInvalidValue;
-    const FdOptions opt{scale, softcap, slopes, window > 0 ? keep_first : 0, sink};
+    if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
+    const FdOptions opt{scale, softcap, slopes, window > 0 ? keep_first : 0, sinks, chunk};
 #define TQ_FD(H)                                                                                                        \
     case H:                                                                                                             \
         return launch_flash_decode<H, FD_SOFTMAX_EXT>((const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages,      \

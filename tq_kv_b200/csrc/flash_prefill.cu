@@ -56,7 +56,8 @@ struct FpSource {
 
 // Options of the EXT form of the kernel: score * scale, capped by softcap * tanh(. / softcap), minus
 // slopes[h] * (query position - key position); behind a window the first keep_first keys stay in view (their
-// tiles are walked first, then the window's); the result times sigmoid(gate[token, h * HD + d]) entry by entry.
+// tiles are walked first, then the window's); with `chunk` (and no window) the query at position p sees the keys
+// p - p % chunk .. p; the result times sigmoid(gate[token, h * HD + d]) entry by entry.
 struct FpOptions {
     float scale;            // natural units
     float softcap;          // > 0: capped scores
@@ -64,7 +65,8 @@ struct FpOptions {
     int keep_first;
     const float* gate;      // float32 logits [T, ldg] (column h * HD + d) or null
     int ldg;
-    int sink;               // != 0: one added to the softmax's denominator (a key of score 0 without a value)
+    const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
+    int chunk;              // > 0: keys of the query's own chunk only
 };
 
 // cap * tanh(x / cap) with 2^x and a fast division (a few ulp; tanh.approx is not enough)
@@ -110,6 +112,13 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
     const int p_first = start + tile * FP_BM;
     const int p_last = start + min(len, tile * FP_BM + FP_BM) - 1;
     int j_begin = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+    int chunk_lo[2] = {0, 0}, chunk_lo_last = 0;           // the first key a row (the tile's last row) sees of its chunk
+    if (EXT && opt.chunk > 0) {
+        j_begin = p_first - p_first % opt.chunk;
+        chunk_lo_last = p_last - p_last % opt.chunk;
+        chunk_lo[0] = rp[0] - rp[0] % opt.chunk;
+        chunk_lo[1] = rp[1] - rp[1] % opt.chunk;
+    }
     j_begin &= ~(FP_BN - 1);
     // kept first tokens that lie in tiles before the window's first: those tiles come first
     const int keep = (EXT && window > 0) ? opt.keep_first : 0;
@@ -190,7 +199,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
         // scale and mask: key j is seen by the row at position p iff p - window < j <= p.  Most tiles lie
         // wholly inside every row's range (the same answer for the whole block): they skip the tests.
         float mx[2] = {-INFINITY, -INFINITY};
-        const bool inside = j0 + FP_BN - 1 <= p_first && (window <= 0 || j0 > p_last - window);
+        const bool inside = j0 + FP_BN - 1 <= p_first && (window <= 0 || j0 > p_last - window) && j0 >= chunk_lo_last;
         if constexpr (EXT) {
             const float slope = opt.slopes ? opt.slopes[h] : 0.f;
             const float tc = opt.softcap > 0.f ? 2.f * 1.4426950408889634f / opt.softcap : 0.f;
@@ -200,7 +209,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
                 for (int e = 0; e < 4; ++e) {
                     const int j = j0 + n * 8 + 2 * tid4 + (e & 1);
                     const int p = rp[e >> 1];
-                    const bool seen = inside || (j <= p && (window <= 0 || j > p - window || j < keep));
+                    const bool seen = inside || (j <= p && j >= chunk_lo[e >> 1] && (window <= 0 || j > p - window || j < keep));
                     float x = s[n][e] * opt.scale;
                     if (opt.softcap > 0.f) x = fp_tanh_cap(x, opt.softcap, tc);
                     x = fmaf(-slope, (float)(p - j), x);
@@ -281,8 +290,8 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         if (ri[r] >= len) continue;
-        // (the sink's share of the denominator is 2^(0 - m) in the units the sums are kept in)
-        const float inv = 1.f / ((EXT && opt.sink) ? l_run[r] + exp2f(-m_run[r]) : l_run[r]);
+        // (the sink's share of the denominator is 2^(sink log2 e - m) in the units the sums are kept in)
+        const float inv = 1.f / ((EXT && opt.sinks) ? l_run[r] + exp2f(fmaf(opt.sinks[h], 1.4426950408889634f, -m_run[r])) : l_run[r]);
         bf16* orow = out + ((size_t)(tok0 + ri[r]) * nh + h) * HD;
         const float* grow = (EXT && opt.gate) ? opt.gate + (size_t)(tok0 + ri[r]) * opt.ldg + (size_t)h * HD : nullptr;
 #pragma unroll
@@ -301,7 +310,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
 template <int HD, bool EXT = false>
 static int launch_flash_prefill(const bf16* q, const FpSource& src, const int* cu_seqlens, const int* start_pos,
                                 int n_seqs, int n_tokens, int window, float scale, bf16* out, int nh, int nkv,
-                                cudaStream_t stream, FpOptions opt = FpOptions{0.f, 0.f, nullptr, 0, nullptr, 0}) {
+                                cudaStream_t stream, FpOptions opt = FpOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0}) {
     constexpr size_t smem = 2 * 2 * FP_BN * (HD * 2 + 16);
     static bool configured = false;
     if (!configured) {
@@ -349,7 +358,7 @@ TQ_API int tq_flash_prefill_ext(const void* q, const void* k_packed, const void*
                                 const void* v_pages, const int* block_table, int table_width, int ring_pages,
                                 int page_tokens, const int* cu_seqlens, const int* start_pos, int n_seqs, int n_tokens,
                                 int window, float scale, float softcap, const float* slopes, int keep_first,
-                                int sink, const float* gate, int ldg, void* out, int nh, int nkv, int hd,
+                                const float* sinks, int chunk, const float* gate, int ldg, void* out, int nh, int nkv, int hd,
                                 cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (nkv <= 0 || nh % nkv || nh > 65535) return (int)cudaErrorNotSupported;
@@ -357,7 +366,8 @@ TQ_API int tq_flash_prefill_ext(const void* q, const void* k_packed, const void*
     if (keep_first < 0 || (keep_first > 0 && !k_packed && ring_pages > 0)) return (int)cudaErrorInvalidValue;
     FpSource src{(const bf16*)k_packed, (const bf16*)v_packed, (const bf16*)k_pages, (const bf16*)v_pages,
                  block_table, table_width, ring_pages, page_tokens};
-    const FpOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sink};
+    if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
+    const FpOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk};
 #define TQ_FP(H)                                                                                                    \
     case H:                                                                                                         \
         return launch_flash_prefill<H, true>((const bf16*)q, src, cu_seqlens, start_pos, n_seqs, n_tokens, window, \

@@ -160,8 +160,8 @@ __device__ __forceinline__ uint64_t ft_desc_mn(uint32_t saddr, uint32_t mn_strid
 // softmax's are.
 // FT_SOFTMAX_EXT: the softmax with options (FtOptions): score * scale, capped by softcap * tanh(. / softcap), minus
 // slopes[h] * (query position - key position); behind a window the first keep_first keys stay in view (the tiles
-// that hold them are walked first, then the window's); the result times sigmoid(gate[token, h * HD + d]) entry by
-// entry.  The scores are transformed in float32 before the maximum is taken.
+// that hold them are walked first, then the window's); with `chunk` (and no window) the query at position p sees
+// the keys p - p % chunk .. p; the result times sigmoid(gate[token, h * HD + d]) entry by entry.  The scores are transformed in float32 before the maximum is taken.
 #define FT_SOFTMAX 0
 #define FT_SIGMOID 1
 #define FT_SOFTMAX_EXT 2
@@ -173,7 +173,8 @@ struct FtOptions {
     int keep_first;
     const float* gate;      // float32 logits [T, ldg] (column h * HD + d) or null
     int ldg;
-    int sink;               // != 0: one added to the softmax's denominator (a key of score 0 without a value)
+    const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
+    int chunk;              // > 0: keys of the query's own chunk only
 };
 
 template <int HD, bool PAGED, int WEIGHTS>
@@ -228,6 +229,11 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const int p_first = start + tile * FT_BM;
     const int p_last = start + min(len, tile * FT_BM + FT_BM) - 1;
     int j_begin = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+    int chunk_lo_last = 0;                                 // the first key the tile's last row sees of its chunk
+    if (WEIGHTS == FT_SOFTMAX_EXT && opt.chunk > 0) {
+        j_begin = p_first - p_first % opt.chunk;
+        chunk_lo_last = p_last - p_last % opt.chunk;
+    }
     j_begin &= ~(FT_BN - 1);
     // kept first tokens that lie in tiles before the window's first: those tiles come first
     const int keep = (WEIGHTS == FT_SOFTMAX_EXT && window > 0) ? opt.keep_first : 0;
@@ -351,6 +357,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         const int r = quarter * 32 + lane;                   // row of the tile = TMEM lane
         const int i_row = tile * FT_BM + r;                  // token index within the sequence
         const int p_row = start + min(i_row, len - 1);       // rows past the end repeat the last row (never stored)
+        const int chunk_lo = (WEIGHTS == FT_SOFTMAX_EXT && opt.chunk > 0) ? p_row - p_row % opt.chunk : 0;
         const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
@@ -373,9 +380,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             if (!ft_wait(ft_smem(&s_full[it & 1]), (it >> 1) & 1, true)) { *failed = 1; ok = false; break; }
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const uint32_t s_addr = tmem_s + (it & 1) * FT_BN + lane_addr;
-            // key j is seen iff p_row - window < j <= p_row; most tiles lie inside every row's range
-            const int j_hi = p_row, j_lo = window > 0 ? p_row - window + 1 : 0;
-            const bool inside = j0 + FT_BN - 1 <= p_first && (window <= 0 || j0 > p_last - window);
+            // key j is seen iff p_row - window < j <= p_row (or chunk_lo <= j <= p_row); most tiles lie inside every row's range
+            const int j_hi = p_row, j_lo = window > 0 ? p_row - window + 1 : chunk_lo;
+            const bool inside = j0 + FT_BN - 1 <= p_first && (window <= 0 || j0 > p_last - window) && j0 >= chunk_lo_last;
             float sv[FT_BN];                                  // the row's scores of this tile
 #pragma unroll
             for (int c = 0; c < FT_BN; c += 32) ft_ld32_issue(s_addr + c, sv + c);
@@ -512,8 +519,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         if (ok) {
             float inv = 1.f / l_run;
-            if constexpr (WEIGHTS == FT_SOFTMAX_EXT) {         // the sink's share: 2^(0 - m_ref), the sums' unit
-                if (opt.sink) inv = 1.f / (l_run + exp2f(-m_ref));
+            if constexpr (WEIGHTS == FT_SOFTMAX_EXT) {         // the sink's share: 2^(sink log2 e - m_ref), the sums' unit
+                if (opt.sinks) inv = 1.f / (l_run + exp2f(fmaf(opt.sinks[h], 1.4426950408889634f, -m_ref)));
             }
             if constexpr (WEIGHTS == FT_SIGMOID)
                 inv = gate ? 1.f / (1.f + expf(-gate[(size_t)(tok0 + min(i_row, len - 1)) * ldg + h])) : 1.f;
@@ -579,7 +586,7 @@ static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
                      int table_width, int ring_pages, const int* cu_seqlens, const int* start_pos, int n_seqs,
                      int n_tokens, int window, float scale, bf16* out, int nh, int nkv, int* status,
                      cudaStream_t stream, const float* bias = nullptr, int n_dist = 0, const float* gate = nullptr,
-                     int ldg = 0, FtOptions opt = FtOptions{0.f, 0.f, nullptr, 0, nullptr, 0}) {
+                     int ldg = 0, FtOptions opt = FtOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0}) {
     constexpr int SMEM = (HD / 64) * (FT_SUB_BYTES + 4 * FT_KV_SUB_BYTES) + 256;
     static bool configured = false;
     if (!configured) {
@@ -671,7 +678,8 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
                                    const void* v_pages, long long n_pages, const int* block_table, int table_width,
                                    int ring_pages, int page_tokens, const int* cu_seqlens, const int* start_pos,
                                    int n_seqs, int n_tokens, int window, float scale, float softcap,
-                                   const float* slopes, int keep_first, int sink, const float* gate, int ldg, void* out, int nh,
+                                   const float* slopes, int keep_first, const float* sinks, int chunk,
+                                   const float* gate, int ldg, void* out, int nh,
                                    int nkv, int hd, int* status, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (nkv <= 0 || nh % nkv || (hd != 64 && hd != 128)) return (int)cudaErrorNotSupported;
@@ -691,7 +699,8 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
         if (!st) st = ft_map(&mv, v_packed, (uint64_t)n_tokens, (uint64_t)nkv * hd, (uint64_t)nkv * hd, FT_BN);
     }
     if (st) return st;
-    const FtOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sink};
+    if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
+    const FtOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk};
 #define TQ_FT(H, P) return ft_launch<H, P, FT_SOFTMAX_EXT>(mq, mk, mv, block_table, table_width, ring_pages, cu_seqlens, \
                                                            start_pos, n_seqs, n_tokens, window, scale, (bf16*)out, nh,    \
                                                            nkv, status, stream, nullptr, 0, nullptr, 0, opt)

@@ -175,6 +175,7 @@ gemv_rows_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const float
                 if (bias) { v0 += bias[n]; if (SWIGLU) v1 += bias[n + N]; }
                 float v = v0;
                 if (SWIGLU) v = gated_act(v0, act) * v1;
+                else if (act == TQ_ACT_SQUARE_RELU) v = square_relu(v0);
                 TO* c = C + (size_t)(m0 + r) * ldc + n;
                 if (accumulate) v += to_f32<TO>(*c);
                 *c = from_f32<TO>(v);
@@ -184,7 +185,8 @@ gemv_rows_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const float
 }
 
 // N is the number of output columns; with swiglu != 0, W has 2*N rows and swiglu names the gate's activation
-// (TQ_ACT_SILU = 1, TQ_ACT_GELU_TANH = 2).
+// (TQ_ACT_SILU = 1, TQ_ACT_GELU_TANH = 2); swiglu == TQ_ACT_SQUARE_RELU (3): a plain product, N rows of W, whose
+// result leaves as the square of its relu.
 TQ_API int tq_gemv_rows(const void* A, int a_dtype, const void* W, int w_dtype, const float* bias, void* C,
                         int c_dtype, int M, int N, int K, int lda, int ldw, int ldc, int accumulate, int swiglu,
                         cudaStream_t stream) {
@@ -194,12 +196,12 @@ TQ_API int tq_gemv_rows(const void* A, int a_dtype, const void* W, int w_dtype, 
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
 #define TQ_LAUNCH2(TA, TW, TO)                                                                                 \
     do {                                                                                                       \
-        if (swiglu)                                                                                            \
+        if (swiglu && swiglu != TQ_ACT_SQUARE_RELU)                                                            \
             gemv_rows_kernel<TA, TW, TO, true><<<grid, GV_WARPS * 32, 0, stream>>>(                           \
                 (const TA*)A, (const TW*)W, bias, (TO*)C, M, N, K, lda, ldw, ldc, accumulate, swiglu);         \
         else                                                                                                   \
             gemv_rows_kernel<TA, TW, TO, false><<<grid, GV_WARPS * 32, 0, stream>>>(                          \
-                (const TA*)A, (const TW*)W, bias, (TO*)C, M, N, K, lda, ldw, ldc, accumulate, 0);              \
+                (const TA*)A, (const TW*)W, bias, (TO*)C, M, N, K, lda, ldw, ldc, accumulate, swiglu);         \
     } while (0)
     const int code = a_dtype * 4 + w_dtype * 2 + c_dtype;
     switch (code) {

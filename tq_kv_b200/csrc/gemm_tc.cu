@@ -52,6 +52,7 @@
 #define EPI_ACCUM 1
 #define EPI_SWIGLU 2
 #define EPI_GELU 3          // as EPI_SWIGLU with the tanh form of gelu on the gate
+#define EPI_RELU2 4         // a plain product (after its bias) through the square of relu
 #define TC_GATED(E) ((E) == EPI_SWIGLU || (E) == EPI_GELU)
 
 // ---- PTX wrappers -------------------------------------------------------------
@@ -170,6 +171,10 @@ __device__ __forceinline__ void tc_epilogue_item(uint32_t t_row, unsigned char* 
             const float mine = col < N ? bias[col] : 0.f;
 #pragma unroll
             for (int j = 0; j < 32; ++j) v[j] += __shfl_sync(0xffffffffu, mine, j);
+        }
+        if (EPI == EPI_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = square_relu(v[j]);
         }
         if (!rows_live) continue;
         unsigned char* pb = st + (piece & 1) * TC_EPI_BYTES;
@@ -706,7 +711,7 @@ static int tc_mode() {
 // A [M, K] and B [N, K] (or [2N, K] with epilogue 2) bfloat16 with row strides
 // lda / ldb (elements, multiples of 8; bases 16-byte aligned); C [M, N] with
 // row stride ldc (base and row stride in bytes multiples of 16), float32 or
-// bfloat16 (epilogue 1 needs float32).
+// bfloat16 (epilogue 1 needs float32, epilogue 4 bfloat16).
 // status: device int, bit 1 is raised if a pipeline wait ran out.
 TQ_API int tq_gemm_tc(const void* A, const void* B, const float* bias, void* C, int c_dtype, int M, int N, int K,
                       int lda, int ldb, int ldc, int epilogue, int* status, cudaStream_t stream) {
@@ -755,6 +760,7 @@ TQ_API int tq_gemm_tc(const void* A, const void* B, const float* bias, void* C, 
     if (epilogue == EPI_SWIGLU && c_dtype == TQ_BF16) TQ_TC(EPI_SWIGLU, bf16);
     if (epilogue == EPI_GELU && c_dtype == TQ_F32) TQ_TC(EPI_GELU, float);
     if (epilogue == EPI_GELU && c_dtype == TQ_BF16) TQ_TC(EPI_GELU, bf16);
+    if (epilogue == EPI_RELU2 && c_dtype == TQ_BF16) TQ_TC(EPI_RELU2, bf16);
 #undef TQ_TC
     return (int)cudaErrorInvalidValue;
 }
@@ -763,7 +769,7 @@ TQ_API int tq_gemm_tc(const void* A, const void* B, const float* bias, void* C, 
 // tile_b_row[i] .. of B (device int32 [ceil(M / 128)]; a negative entry: the tile is skipped and its rows of
 // C stay as they are).  B [b_rows, K] stacks the groups' matrices; with epilogue 2 a group's block holds its
 // gate rows and, b_rows_second rows further on, its up rows.  C [M, N]: columns past N are never written, so a
-// tile may reach into the next group's rows of B.  Epilogues 0 (store) and 2 (SwiGLU); other rules as tq_gemm_tc.
+// tile may reach into the next group's rows of B.  Epilogues 0 (store), 2 (SwiGLU) and, bfloat16, 4 (squared relu); other rules as tq_gemm_tc.
 TQ_API int tq_gemm_tc_grouped(const void* A, const void* B, void* C, int c_dtype, int M, int N, int K, int lda, int ldb,
                               int ldc, int epilogue, int b_rows, int b_rows_second, const int* tile_b_row, int* status,
                               cudaStream_t stream) {
@@ -774,7 +780,8 @@ TQ_API int tq_gemm_tc_grouped(const void* A, const void* B, void* C, int c_dtype
     if (c_dtype != TQ_F32 && c_dtype != TQ_BF16) return (int)cudaErrorInvalidValue;
     if ((reinterpret_cast<uintptr_t>(C) & 15) || ((size_t)ldc * (c_dtype == TQ_F32 ? 4 : 2)) % 16)
         return (int)cudaErrorInvalidValue;
-    if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU) return (int)cudaErrorInvalidValue;
+    if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU && !(epilogue == EPI_RELU2 && c_dtype == TQ_BF16))
+        return (int)cudaErrorInvalidValue;
     CUtensorMap ma, mb, mc;
     int st = make_map(&ma, A, (uint64_t)M, (uint64_t)K, (uint64_t)lda, TC_BM);
     if (st) return st;
@@ -784,6 +791,8 @@ TQ_API int tq_gemm_tc_grouped(const void* A, const void* B, void* C, int c_dtype
     if (st) return st;
     if (epilogue == EPI_STORE && c_dtype == TQ_F32)
         return launch_tc_grouped<EPI_STORE, float>(ma, mb, mc, M, N, K, 0, tile_b_row, status, stream);
+    if (epilogue == EPI_RELU2)
+        return launch_tc_grouped<EPI_RELU2, bf16>(ma, mb, mc, M, N, K, 0, tile_b_row, status, stream);
     if (epilogue == EPI_STORE)
         return launch_tc_grouped<EPI_STORE, bf16>(ma, mb, mc, M, N, K, 0, tile_b_row, status, stream);
     if (c_dtype == TQ_F32)

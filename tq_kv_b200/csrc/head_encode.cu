@@ -12,8 +12,10 @@
 //   `row_inv` (float32 [T, 2]: one factor per token for its whole q row and
 //   one for its whole k row, made by row_inv_rms below) and weights over those
 //   whole rows, q and k are first multiplied by factor * weight: an RMS norm
-//   over the whole projection, before the heads are split and turned;
-//   v heads (vd entries each) are copied: from their own columns, or — v_col < 0
+//   over the whole projection, before the heads are split and turned; with
+//   norm_eps and weights of one head's size (shared by the heads) each head is
+//   normed, weighted and then turned;
+//   v heads (vd entries each) are copied, times v_scale: from their own columns, or — v_col < 0
 //   — from the k columns as projected, before the rotation (vd == hd then).
 //
 // q goes to q_out [T, nh*hd]; k and v go to the packed outputs (if given) and
@@ -37,7 +39,7 @@ head_encode_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col,
                    int ring_pages, int page_tokens, TC* __restrict__ q_out, TC* __restrict__ k_out,
                    TC* __restrict__ v_out, TC* __restrict__ k_pages, TC* __restrict__ v_pages, int nh, int nkv,
                    int hd, int vd, const float* __restrict__ row_inv, const float* __restrict__ q_w,
-                   const float* __restrict__ k_w, int paired) {
+                   const float* __restrict__ k_w, int paired, float v_scale) {
     // grid (token, groups of four heads), a warp per head: heads 0..nh-1 are q, then nkv k heads, then nkv v heads
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int head = blockIdx.y * 4 + (threadIdx.x >> 5);
@@ -71,7 +73,7 @@ head_encode_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col,
     pdl_launch();
     if (!is_q && !is_k) {                                    // values: a copy
         for (int d = lane; d < width; d += 32) {
-            const TC r = from_f32<TC>(x[d]);
+            const TC r = from_f32<TC>(x[d] * v_scale);
             if (dst) dst[d] = r;
             if (cache) cache[d] = r;
         }
@@ -84,10 +86,10 @@ head_encode_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col,
         ss = warp_sum(ss);
         inv = 1.f / sqrtf(ss / (float)width + norm_eps);
     }
-    const float* w = nullptr;                                // the whole-row norm's weights of this head
+    const float* w = is_q ? q_w : k_w;                       // the norm's weights: of every head, or (whole-row norm) of this one
     if (row_inv) {
         inv = row_inv[2 * t + (is_q ? 0 : 1)];
-        w = (is_q ? q_w : k_w) + (size_t)g * hd;
+        w += (size_t)g * hd;
     }
     const int half = rot >> 1;
     if (half > 0) {
@@ -116,9 +118,10 @@ TQ_API int tq_head_encode(const float* proj, int ld, int q_col, int k_col, int v
                           const int* new_lens, const int* block_table, int table_width, int ring_pages,
                           int page_tokens, void* q_out, void* k_out, void* v_out, void* k_pages, void* v_pages,
                           int cache_dtype, int n_tokens, int nh, int nkv, int hd, int vd, const float* row_inv,
-                          const float* q_w, const float* k_w, int paired, cudaStream_t stream) {
+                          const float* q_w, const float* k_w, int paired, float v_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (row_inv && (!q_w || (nkv > 0 && !k_w) || norm_eps > 0.f)) return (int)cudaErrorInvalidValue;
+    if ((q_w || k_w) && !row_inv && !(norm_eps > 0.f)) return (int)cudaErrorInvalidValue;
     if (rot < 0 || rot > hd || (rot & 1) || page_tokens <= 0 || hd <= 0 || vd <= 0) return (int)cudaErrorInvalidValue;
     if (rot > 0 && (!cos_tab || !sin_tab)) return (int)cudaErrorInvalidValue;
     if ((k_pages == nullptr) != (v_pages == nullptr)) return (int)cudaErrorInvalidValue;
@@ -131,7 +134,7 @@ TQ_API int tq_head_encode(const float* proj, int ld, int q_col, int k_col, int v
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, head_encode_kernel<TC>, grid, dim3(128), 0, stream, proj, ld, q_col,  \
                          k_col, v_col, cos_tab, sin_tab, rot, norm_eps, tok_pos, tok_seq, new_lens, block_table,   \
                          table_width, ring_pages, page_tokens, (TC*)q_out, (TC*)k_out, (TC*)v_out, (TC*)k_pages,   \
-                         (TC*)v_pages, nh, nkv, hd, vd, row_inv, q_w, k_w, paired)
+                         (TC*)v_pages, nh, nkv, hd, vd, row_inv, q_w, k_w, paired, v_scale)
     if (cache_dtype == TQ_F32) TQ_LAUNCH(float);
     if (cache_dtype == TQ_BF16) TQ_LAUNCH(bf16);
 #undef TQ_LAUNCH

@@ -3,6 +3,8 @@
 // and a token's result is the mean of its experts' results, or their sum with a weight per (token, expert)
 // where a router gives weights (router_choice below).
 //
+// Experts without a gate, W_down[e] max(W_up[e] x, 0)^2, are the same with w_up [E, F, W] in w_gu's place.
+//
 // The experts' weights are stacked: w_gu [E, 2*F, W] (an expert's gate rows, then its up rows) and
 // w_down [E, W, F].  choice [T, top] int32 names each token's experts.
 //
@@ -83,6 +85,101 @@ TQ_API int tq_router_choice(const float* logits, int ld, int n_experts, int top,
                          ld, n_experts, top, scale, floor_, choice, weights, n_tokens);
 }
 
+// ---- choice with groups --------------------------------------------------------------------------------------
+// scores s = softmax(logits) over all experts; the choice goes by c = s + correction (null: s alone).  The experts
+// lie in n_groups equal groups of neighbours; a group counts as its largest c, and only experts of the `keep` best
+// groups can be chosen.  Of those the `top` with the largest c are (the lowest index first among equals, of groups
+// too); their weights are their s as they are.  A warp per token; float32 throughout.
+__device__ __forceinline__ void warp_best(float& best, int& best_i, int none) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, best_i, o);
+        if (oi < none && (best_i == none || ob > best || (ob == best && oi < best_i))) { best = ob; best_i = oi; }
+    }
+}
+
+__global__ void __launch_bounds__(128)
+group_router_choice_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int n_experts,
+                           int top, int n_groups, int keep, int* __restrict__ choice, float* __restrict__ weights,
+                           int n_tokens) {
+    extern __shared__ float router_sh[];                  // per warp: s [E], c [E], group scores [n_groups]
+    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= n_tokens) return;
+    float* s = router_sh + (threadIdx.x >> 5) * (2 * n_experts + n_groups);
+    float* c = s + n_experts;
+    float* gs = c + n_experts;
+    const int per = n_experts / n_groups;
+    pdl_wait();
+    pdl_launch();
+    const float* z = logits + (size_t)t * ld;
+    float m = -INFINITY;
+    for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    float sum = 0.f;
+    for (int e = lane; e < n_experts; e += 32) {
+        const float p = expf(z[e] - m);
+        s[e] = p;
+        sum += p;
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < n_experts; e += 32) {
+        s[e] /= sum;
+        c[e] = s[e] + (correction ? correction[e] : 0.f);
+    }
+    __syncwarp();
+    if (keep < n_groups) {
+        for (int g = lane; g < n_groups; g += 32) {
+            float best = c[g * per];
+            for (int i = 1; i < per; ++i) best = fmaxf(best, c[g * per + i]);
+            gs[g] = best;
+        }
+        __syncwarp();
+        // the keep best groups are marked by +inf, one after the other; the experts of all others leave the choice
+        for (int k = 0; k < keep; ++k) {
+            float best = 0.f;
+            int best_g = n_groups;
+            for (int g = lane; g < n_groups; g += 32)
+                if (gs[g] < INFINITY && (best_g == n_groups || gs[g] > best)) { best = gs[g]; best_g = g; }
+            warp_best(best, best_g, n_groups);
+            __syncwarp();
+            if (lane == 0 && best_g < n_groups) gs[best_g] = INFINITY;
+            __syncwarp();
+        }
+        for (int e = lane; e < n_experts; e += 32)
+            if (gs[e / per] < INFINITY) c[e] = -INFINITY;
+        __syncwarp();
+    }
+    for (int k = 0; k < top; ++k) {
+        float best = 0.f;
+        int best_e = n_experts;
+        for (int e = lane; e < n_experts; e += 32)
+            if (c[e] > -INFINITY && (best_e == n_experts || c[e] > best)) { best = c[e]; best_e = e; }
+        warp_best(best, best_e, n_experts);
+        if (best_e >= n_experts) best_e = 0;              // (scores that are no numbers choose nothing)
+        __syncwarp();
+        if (lane == 0) {
+            choice[t * top + k] = best_e;
+            weights[t * top + k] = s[best_e];
+            c[best_e] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
+TQ_API int tq_group_router_choice(const float* logits, int ld, const float* correction, int n_experts, int top,
+                                  int n_groups, int keep, int* choice, float* weights, int n_tokens,
+                                  cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (!logits || !choice || !weights || n_groups < 1 || n_experts % n_groups || keep < 1 || keep > n_groups || top < 1 ||
+        top > keep * (n_experts / n_groups))
+        return (int)cudaErrorInvalidValue;
+    const size_t smem = (size_t)4 * (2 * n_experts + n_groups) * sizeof(float);
+    if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, group_router_choice_kernel, dim3((n_tokens + 3) / 4), dim3(128), smem, stream,
+                         logits, ld, correction, n_experts, top, n_groups, keep, choice, weights, n_tokens);
+}
+
 // ---- a warp's inner product over n entries ---------------------------------------------------------------------
 template <typename TA, typename TB>
 __device__ __forceinline__ float warp_dot(const TA* __restrict__ a, const TB* __restrict__ b, int n, bool vec) {
@@ -105,7 +202,8 @@ __device__ __forceinline__ float warp_dot(const TA* __restrict__ a, const TB* __
 }
 
 // grid (T*top, ceil(F / 8)), 8 warps: warp w computes entry i = blockIdx.y*8 + w
-template <typename TX, typename TW, typename TO>
+// (GATED false: w_gu holds F up rows per expert, the entry is max(up . x, 0)^2)
+template <typename TX, typename TW, typename TO, bool GATED>
 __global__ void __launch_bounds__(256)
 routed_gate_up_kernel(const TX* __restrict__ x, int ldx, const TW* __restrict__ w_gu, const int* __restrict__ choice,
                       int top, int W, int F, TO* __restrict__ act, bool vec) {
@@ -116,8 +214,12 @@ routed_gate_up_kernel(const TX* __restrict__ x, int ldx, const TW* __restrict__ 
     pdl_launch();
     const int e = choice[pair];
     const TX* xr = x + (size_t)(pair / top) * ldx;
-    const TW* wg = w_gu + ((size_t)e * 2 * F + i) * W;
+    const TW* wg = w_gu + ((size_t)e * (GATED ? 2 : 1) * F + i) * W;
     const float g = warp_dot<TX, TW>(xr, wg, W, vec);
+    if (!GATED) {
+        if ((threadIdx.x & 31) == 0) act[(size_t)pair * F + i] = from_f32<TO>(square_relu(g));
+        return;
+    }
     const float u = warp_dot<TX, TW>(xr, wg + (size_t)F * W, W, vec);
     if ((threadIdx.x & 31) == 0) act[(size_t)pair * F + i] = from_f32<TO>(g / (1.f + expf(-g)) * u);
 }
@@ -149,9 +251,10 @@ routed_down_kernel(const TA* __restrict__ act, const TW* __restrict__ w_down, co
 static inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 // x [T, W] (row stride ldx), act [T*top, F] of x's dtype (scratch), y [T, W] float32.  Weights float32 or bfloat16.
+// gated 0: experts without a gate, w_gu [E, F, W].
 TQ_API int tq_routed_experts_rows(const void* x, int x_dtype, int ldx, const void* w_gu, const void* w_down, int w_dtype,
                                   const int* choice, const float* weights, int top, int n_tokens, int W, int F,
-                                  void* act, float* y, int accumulate, cudaStream_t stream) {
+                                  void* act, float* y, int accumulate, int gated, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top < 1 || W <= 0 || F <= 0) return (int)cudaErrorInvalidValue;
     const int xs = x_dtype == TQ_BF16 ? 2 : 4, ws = w_dtype == TQ_BF16 ? 2 : 4;
@@ -162,8 +265,10 @@ TQ_API int tq_routed_experts_rows(const void* x, int x_dtype, int ldx, const voi
     if (g1.y > 65535 || g2.y > 65535) return (int)cudaErrorInvalidValue;
     int st;
 #define TQ_RUN(TX, TW)                                                                                                \
-    st = tq_launch_pdl(TQ_PDL_ELEMENTWISE, routed_gate_up_kernel<TX, TW, TX>, g1, dim3(256), 0, stream, (const TX*)x, \
-                       ldx, (const TW*)w_gu, choice, top, W, F, (TX*)act, vec_up);                                   \
+    st = gated ? tq_launch_pdl(TQ_PDL_ELEMENTWISE, routed_gate_up_kernel<TX, TW, TX, true>, g1, dim3(256), 0, stream, \
+                               (const TX*)x, ldx, (const TW*)w_gu, choice, top, W, F, (TX*)act, vec_up)              \
+               : tq_launch_pdl(TQ_PDL_ELEMENTWISE, routed_gate_up_kernel<TX, TW, TX, false>, g1, dim3(256), 0, stream, \
+                               (const TX*)x, ldx, (const TW*)w_gu, choice, top, W, F, (TX*)act, vec_up);             \
     if (st) return st;                                                                                                \
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, routed_down_kernel<TX, TW>, g2, dim3(256), 0, stream, (const TX*)act,   \
                          (const TW*)w_down, choice, weights, top, W, F, y, accumulate, vec_down)

@@ -12,7 +12,8 @@
 //     its vectors to be scaled to unit length, x * scale / sqrt(sum(x^2) + eps);
 //   * the per-token scalars of a recurrence with one decay per head:  with sp = softplus(raw[t, h] + dt_bias[h]),
 //     g = exp(-exp(A_log[h]) * sp), and second = sigmoid(beta_raw[t, h]) if given, else sp.  They are written as
-//     [T, H, 4] floats (g, second, 0, 0), the layout the scan kernels stage with 16-byte copies.
+//     [T, H, 4] floats (g, second, 0, 0), the layout the scan kernels stage with 16-byte copies.  A recurrence
+//     whose decays are made elsewhere gives beta_raw alone (g is then 1).
 //
 // A warp owns one (token, vector); a lane holds up to CONV_MAX_PER_LANE of its channels.  Steps in which every
 // sequence brings one token shift the state in the same kernel; otherwise a second, small kernel (a thread per
@@ -59,8 +60,11 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ConvArgs a) {
         const long long idx = (long long)(warp_global - n_rows) * 32 + lane;
         if (a.H > 0 && idx < (long long)a.T * a.H) {
             const int t = (int)(idx / a.H), h = (int)(idx - (long long)t * a.H);
-            const float sp = conv_softplus(a.gate_raw[(size_t)t * a.ldg + h] + a.dt_bias[h]);
-            const float g = expf(-expf(a.A_log[h]) * sp);
+            float sp = 0.f, g = 1.f;                     // (no decay per head: the write strength alone)
+            if (a.gate_raw) {
+                sp = conv_softplus(a.gate_raw[(size_t)t * a.ldg + h] + a.dt_bias[h]);
+                g = expf(-expf(a.A_log[h]) * sp);
+            }
             const float second = a.beta_raw ? 1.f / (1.f + expf(-a.beta_raw[(size_t)t * a.ldb + h])) : sp;
             *reinterpret_cast<float4*>(a.scal + (size_t)idx * 4) = make_float4(g, second, 0.f, 0.f);
         }
@@ -150,7 +154,7 @@ __global__ void short_conv_state_kernel(ConvArgs a, int n_seqs) {
         if (r < K - 1) st[(size_t)r * C + c] = keep[r];
 }
 
-// regions: n_reg rows of (first, count, width, unit) ints and the scales as floats.  gate_raw == null: no scalars.
+// regions: n_reg rows of (first, count, width, unit) ints and the scales as floats.  gate_raw and beta_raw null: no scalars.
 TQ_API int tq_short_conv(const float* x, int ldx, const float* w, const float* bias, float* out, int ldo, float* state,
                          long long state_stride, const int* tok_seq, const int* cu_seqlens, const int* slots,
                          int n_seqs, int n_tokens, int C, int K, int silu, int single, int n_reg, const int* regions,
@@ -178,8 +182,8 @@ TQ_API int tq_short_conv(const float* x, int ldx, const float* w, const float* b
     }
     a.n_vec = n_vec;
     long long warps = (long long)n_tokens * n_vec;
-    if (gate_raw) {
-        if (!A_log || !dt_bias || !scal || H <= 0) return (int)cudaErrorInvalidValue;
+    if (gate_raw || beta_raw) {
+        if ((gate_raw && (!A_log || !dt_bias)) || !scal || H <= 0) return (int)cudaErrorInvalidValue;
         a.gate_raw = gate_raw; a.ldg = ldg; a.beta_raw = beta_raw; a.ldb = ldb; a.A_log = A_log; a.dt_bias = dt_bias;
         a.scal = scal; a.H = H;
         warps += ((long long)n_tokens * H + 31) / 32;

@@ -47,8 +47,9 @@ __device__ __forceinline__ uint4 ld_stream16(const void* p) {
 // x = bfloat16(h * g) and scales each batch row's sums by 1 / sqrt(mean(h^2) + eps) before the epilogue, so
 // that the norm needs no kernel and no trip through memory of its own.  The sums of squares are gathered
 // beside the partial products (every k is read by exactly one lane of one warp of one block of the cluster).
-// The gate's activation of a gated product (TQ_ACT_*): the exported functions set it from their `swiglu` argument
-// (1 or 2; 0: not gated) right before they launch, on the launching thread.
+// The gate's activation of a gated product (TQ_ACT_*), or TQ_ACT_SQUARE_RELU on a plain one: the exported functions
+// set it from their `swiglu` argument (1 or 2: gated; 3: plain, squared relu; 0: plain) right before they launch, on
+// the launching thread.
 static thread_local int sk_gate_act = TQ_ACT_SILU;
 
 template <int NT, int TW, bool SWIGLU, typename TO, bool NORM>
@@ -233,6 +234,8 @@ skinny_gemm_kernel(const void* __restrict__ Xv, const bf16* __restrict__ W, cons
             if (bias) { v += bias[col]; if (SWIGLU) u += bias[col + N]; }
             if (SWIGLU)                // (a bfloat16 result keeps 8 bits: the fast exponential and division do)
                 v = (sizeof(TO) == 2 ? gated_act_fast(v, act) : gated_act(v, act)) * u;
+            else if (act == TQ_ACT_SQUARE_RELU)
+                v = square_relu(v);
             TO* y = Y + (size_t)m * ldy + col;
             if (accumulate) v += to_f32<TO>(*y);
             *y = from_f32<TO>(v);
@@ -302,8 +305,10 @@ TQ_API int tq_skinny_gemm(const void* X, const void* W, const float* bias, void*
     if ((reinterpret_cast<uintptr_t>(X) & 15) || (reinterpret_cast<uintptr_t>(W) & 15))
         return (int)cudaErrorInvalidValue;
     if (accumulate && y_dtype != TQ_F32) return (int)cudaErrorInvalidValue;
-    if (swiglu != 0 && swiglu != TQ_ACT_SILU && swiglu != TQ_ACT_GELU_TANH) return (int)cudaErrorInvalidValue;
+    if (swiglu < 0 || swiglu > TQ_ACT_SQUARE_RELU || (swiglu == TQ_ACT_SQUARE_RELU && accumulate))
+        return (int)cudaErrorInvalidValue;
     sk_gate_act = swiglu ? swiglu : TQ_ACT_SILU;
+    if (swiglu == TQ_ACT_SQUARE_RELU) swiglu = 0;
     const bf16* x = (const bf16*)X;
     const bf16* w = (const bf16*)W;
     if (swiglu) {

@@ -7,12 +7,23 @@
 // One kernel does both ends of a sublayer boundary for a token: it applies the
 // write of the sublayer that has just finished (if any) and prepares the input
 // of the next reader (if any): u, and optionally its RMS norm
-// u / sqrt(mean(u^2) + eps) * w, in the dtype the reader wants.  So a layer of
+// u / sqrt(mean(u^2) + eps) * w, in the dtype the reader wants.  Instead of that
+// norm the reader may ask for one without statistics, tanh(alpha * u) * w + b,
+// and y may enter times a vector (a layer's scale) and times sigmoid of a row of
+// gate logits (StreamExtras).  So a layer of
 // two sublayers costs two launches, and the sum of the streams that the final
 // norm reads is the same kernel with read = 1.  All sums are float32.
 #include "common.cuh"
 
 #define SM_MAX_STREAMS 8
+
+struct StreamExtras {
+    const float* y_scale;    // [W] or null: y enters times it, entry by entry
+    const float* y_gate;     // float32 logits [T, ldg] or null: ... and times sigmoid(y_gate[t, i])
+    int ldg;
+    const float* alpha;      // one number or null: the norm is tanh(alpha * u) * norm_w + norm_b
+    const float* norm_b;     // [W]
+};
 
 struct StreamCoefs {
     float mix[SM_MAX_STREAMS * SM_MAX_STREAMS];
@@ -29,7 +40,7 @@ __global__ void __launch_bounds__(256, NS <= 3 ? 4 : (NS == 4 ? 3 : 1))
 streams_step_kernel(float* __restrict__ xs, int S_any, int T, int W, const float* __restrict__ y,
                     const float* __restrict__ mix, const float* __restrict__ write, const float* __restrict__ read,
                     const float* __restrict__ norm_w, float eps, TO* __restrict__ out,
-                    const int* __restrict__ rows) {
+                    const int* __restrict__ rows, StreamExtras ex) {
     const int S = NS < SM_MAX_STREAMS ? NS : S_any;
     extern __shared__ float u_sh[];
     __shared__ float red[32];
@@ -42,9 +53,11 @@ streams_step_kernel(float* __restrict__ xs, int S_any, int T, int W, const float
         cf.write[threadIdx.x] = write ? write[threadIdx.x] : 0.f;
         cf.read[threadIdx.x] = read ? read[threadIdx.x] : 0.f;
     }
+    const float alpha = ex.alpha ? *ex.alpha : 0.f;
     pdl_wait();
     pdl_launch();
     __syncthreads();
+    TO* o_row = out + (size_t)r * W;
     const size_t stride = (size_t)T * W;
     float* row = xs + (size_t)t * W;
     float ss = 0.f;
@@ -67,6 +80,23 @@ streams_step_kernel(float* __restrict__ xs, int S_any, int T, int W, const float
                 yv[0] = v.x; yv[1] = v.y; yv[2] = v.z; yv[3] = v.w;
             } else {
                 yv[0] = y[(size_t)t * W + i];
+            }
+            if (ex.y_scale) {
+                if constexpr (VEC == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(ex.y_scale + i);
+                    yv[0] *= v.x; yv[1] *= v.y; yv[2] *= v.z; yv[3] *= v.w;
+                } else {
+                    yv[0] *= ex.y_scale[i];
+                }
+            }
+            if (ex.y_gate) {
+                const float* gp = ex.y_gate + (size_t)t * ex.ldg + i;
+                if constexpr (VEC == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(gp);
+                    yv[0] /= 1.f + expf(-v.x); yv[1] /= 1.f + expf(-v.y); yv[2] /= 1.f + expf(-v.z); yv[3] /= 1.f + expf(-v.w);
+                } else {
+                    yv[0] /= 1.f + expf(-*gp);
+                }
             }
             float nx[NS][VEC];
 #pragma unroll
@@ -94,7 +124,23 @@ streams_step_kernel(float* __restrict__ xs, int S_any, int T, int W, const float
                         row[s * stride + i] = x[s][0];
                 }
         }
-        if (out) {
+        if (out && ex.alpha) {                       // entry by entry: nothing to gather over the row
+            float n[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                float u = 0.f;
+#pragma unroll
+                for (int s = 0; s < NS; ++s)
+                    if (s < S) u = fmaf(cf.read[s], x[s][e], u);
+                n[e] = fmaf(tanhf(alpha * u), norm_w[i + e], ex.norm_b[i + e]);
+            }
+            if constexpr (VEC == 4) {
+                store2_f32<TO>(o_row + i, n[0], n[1]);
+                store2_f32<TO>(o_row + i + 2, n[2], n[3]);
+            } else {
+                o_row[i] = from_f32<TO>(n[0]);
+            }
+        } else if (out) {
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
                 float u = 0.f;
@@ -106,11 +152,11 @@ streams_step_kernel(float* __restrict__ xs, int S_any, int T, int W, const float
             }
         }
     }
-    if (!out) return;
+    if (!out || ex.alpha) return;
     float inv = 1.f;
     if (norm_w) inv = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
     // (each thread reads back only what it wrote itself)
-    TO* o = out + (size_t)r * W;
+    TO* o = o_row;
     for (int i = threadIdx.x * VEC; i < W; i += blockDim.x * VEC) {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
@@ -122,20 +168,28 @@ streams_step_kernel(float* __restrict__ xs, int S_any, int T, int W, const float
 
 // xs: [S, T, W] float32.  y: [T, W] float32 or null.  mix [S, S], write [S], read [S], norm_w [W]: float32 or
 // null.  out: [n_rows, W] of out_dtype or null.  rows: int32 [n_rows] or null (then n_rows == T); with rows
-// given the streams are not changed: the write is applied on the way to `out` only.
+// given the streams are not changed: the write is applied on the way to `out` only.  y_scale [W], y_gate [T, ldg],
+// alpha (one number), norm_b [W]: see StreamExtras; float32 or null.
 TQ_API int tq_streams_step(float* xs, int S, int T, int W, const float* y, const float* mix, const float* write,
                            const float* read, const float* norm_w, float eps, void* out, int out_dtype,
-                           const int* rows, int n_rows, cudaStream_t stream) {
+                           const int* rows, int n_rows, const float* y_scale, const float* y_gate, int ldg,
+                           const float* alpha, const float* norm_b, cudaStream_t stream) {
     if (n_rows <= 0 || T <= 0) return 0;
     if (S < 1 || S > SM_MAX_STREAMS || W <= 0 || W > 12288) return (int)cudaErrorInvalidValue;
     if (y && (!mix || !write)) return (int)cudaErrorInvalidValue;
     if (out && !read) return (int)cudaErrorInvalidValue;
     if (!y && !out) return 0;
-    const size_t smem = out ? (size_t)W * sizeof(float) : 0;
-    const bool vec = (W % 4 == 0) && ((reinterpret_cast<uintptr_t>(xs) | reinterpret_cast<uintptr_t>(y)) % 16 == 0);
+    if (alpha && (!norm_w || !norm_b)) return (int)cudaErrorInvalidValue;
+    if ((y_scale || y_gate) && !y) return (int)cudaErrorInvalidValue;
+    if (y_gate && ldg < W) return (int)cudaErrorInvalidValue;
+    const StreamExtras ex{y_scale, y_gate, ldg, alpha, norm_b};
+    const size_t smem = out && !alpha ? (size_t)W * sizeof(float) : 0;
+    const bool vec = (W % 4 == 0) && (!y_gate || ldg % 4 == 0) &&
+                     ((reinterpret_cast<uintptr_t>(xs) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(y_scale) |
+                       reinterpret_cast<uintptr_t>(y_gate) | reinterpret_cast<uintptr_t>(out)) % 16 == 0);
 #define TQ_LAUNCH_NS(TO, V, NS)                                                                                  \
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, streams_step_kernel<TO, V, NS>, dim3(n_rows), dim3(256), smem,      \
-                         stream, xs, S, T, W, y, mix, write, read, norm_w, eps, (TO*)out, rows)
+                         stream, xs, S, T, W, y, mix, write, read, norm_w, eps, (TO*)out, rows, ex)
 #define TQ_LAUNCH(TO, V)                                                                                         \
     switch (S) {                                                                                                 \
         case 1: TQ_LAUNCH_NS(TO, V, 1);                                                                          \

@@ -129,7 +129,7 @@ class DecoderModel:
         if batch.n_logit_rows == 0:
             return None
         if isinstance(h, ResidualStreams):
-            normed = h.read_sum(self.final_norm.weight, self.final_norm.eps, rt.act_dtype, rows=batch.logit_rows)
+            normed = h.read_sum(self.final_norm.stream_args(), rt.act_dtype, rows=batch.logit_rows)
         else:
             normed = self.final_norm.forward(h, rt.act_dtype, rows=batch.logit_rows)
         logits = self.head.forward(normed)

@@ -174,14 +174,18 @@ _SIGNATURES = {
     "tq_flash_prefill_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int,
                             c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int,
                             c_void_p, c_void_p],
-    "tq_attention_merge": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "tq_attention_merge": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "tq_embed_sinusoid": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "tq_group_rmsnorm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int,
                          c_float, c_int, c_void_p],
     "tq_embed_scaled": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
+    "tq_square_relu": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "tq_add_scaled": [c_void_p, c_void_p, c_size_t, c_float, c_void_p],
     "tq_gated_scan": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, ctypes.c_longlong,
                       c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "tq_channel_delta_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
+                              ctypes.c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                              c_int, c_void_p],
     "tq_short_conv": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, ctypes.c_longlong, c_void_p,
                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                       c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
@@ -215,19 +219,19 @@ _SIGNATURES = {
     "tq_sigmoid_attention_sum": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "tq_attention_ext": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p,
-                         c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+                         c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
     "tq_flash_prefill_tc_ext": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int,
                                 c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p,
-                                c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+                                c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "tq_flash_prefill_ext": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                             c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_int, c_void_p,
+                             c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p,
                              c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "tq_flash_decode_ext": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
-                            c_float, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                            c_float, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                             c_int, c_int, c_void_p],
     "tq_head_encode": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                       c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                       c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p],
     "tq_row_inv_rms": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "tq_add_normed_copy": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "tq_round_rows": [c_void_p, c_void_p, c_size_t, c_void_p],
@@ -239,11 +243,18 @@ _SIGNATURES = {
     "tq_sigmoid_gate": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "tq_tanh_cap": [c_void_p, c_size_t, c_float, c_void_p],
     "tq_streams_step": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
-                        c_void_p, c_int, c_void_p, c_int, c_void_p],
+                        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
     "tq_streams_fill": [c_void_p, c_void_p, c_int, c_size_t, c_void_p],
     "tq_table_choice": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
     "tq_routed_experts_rows": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                               c_int, c_void_p, c_void_p, c_int, c_void_p],
+                               c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
+    "tq_group_router_choice": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p],
+    "tq_gru_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_int, c_int,
+                    c_int, c_float, c_void_p, c_int, c_void_p],
+    "tq_low_rank_rows": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                         c_void_p, c_int, c_int, c_int, c_void_p],
+    "tq_channel_decay": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "tq_round_columns": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
     "tq_routed_sort": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                        c_void_p, c_void_p, c_void_p, c_void_p],
     "tq_routed_combine": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p],

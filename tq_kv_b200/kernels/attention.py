@@ -134,15 +134,17 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
                   k_pages: Optional[torch.Tensor] = None, v_pages: Optional[torch.Tensor] = None,
                   block_table: Optional[torch.Tensor] = None, table_width: int = 0, ring_pages: int = 0,
                   page_tokens: int = 64, n_splits: int = 1, scratch: Optional[torch.Tensor] = None,
-                  gate: Optional[torch.Tensor] = None, use_fast: bool = True, sink: bool = False):
+                  gate: Optional[torch.Tensor] = None, use_fast: bool = True, sink=False,
+                  chunk: Optional[int] = None):
     """Softmax attention with options: for the query at position i of head h and the key at position j <= i,
 
         s = q . k * scale;   s <- softcap * tanh(s / softcap)  (if a cap is given);
         s <- s - slopes[h] * (i - j)                            (if slopes are given);
 
-    j is visible if i - j < window or j < keep_first (no window: every j <= i).  With `sink` the softmax's
-    denominator counts one more key of score 0 that has no value: p_j = exp(s_j) / (1 + sum exp(s)).  Value rows may have another
-    width than the keys.  q [T, nh*key_dim], out [T, nh*value_dim]; keys and values as in `attention`.
+    j is visible if i - j < window or j < keep_first (no window: every j <= i); with `chunk` (and no window) if
+    i // chunk == j // chunk.  `sink`: a float32 tensor [n_heads] — the softmax's denominator counts one more key of
+    score sink[h] that has no value, p_j = exp(s_j) / (exp(sink[h]) + sum exp(s)) — or True (a score of 0) or False.
+    Value rows may have another width than the keys.  q [T, nh*key_dim], out [T, nh*value_dim]; keys and values as in `attention`.
     `gate` (float32 [T, nh*value_dim], possibly a column slice of wider rows): out *= sigmoid(gate), in the
     attention kernel's last step where it can, else by a kernel of its own.
 
@@ -168,6 +170,14 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
         raise KernelError("attention: slopes must be float32 [n_heads]")
     if keep_first and ring_pages:
         raise KernelError("attention: kept first tokens need a cache that keeps all keys")
+    if chunk and window:
+        raise KernelError("attention: a window or chunks, not both")
+    if sink is True:
+        sink = torch.zeros(n_heads, dtype=torch.float32, device=q.device)
+    elif sink is False:
+        sink = None
+    if sink is not None and (sink.dtype != torch.float32 or tuple(sink.shape) != (n_heads,)):
+        raise KernelError("attention: sink must be float32 [n_heads]")
     part_acc = part_ml = None
     if n_splits > 1:
         need = split_scratch_floats(T, n_heads, value_dim, n_splits)
@@ -176,7 +186,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
         n_acc = T * n_heads * n_splits * value_dim
         part_acc, part_ml = scratch[:n_acc], scratch[n_acc:need]
     need_contiguous(q=q, out=out, k_packed=k_packed, v_packed=v_packed, k_pages=k_pages, v_pages=v_pages,
-                    block_table=block_table, slopes=slopes)
+                    block_table=block_table, slopes=slopes, sink=sink)
     if gate is not None and (gate.dtype != torch.float32 or tuple(gate.shape) != tuple(out.shape)
                              or gate.stride(1) != 1):
         raise KernelError("attention: the gate must be float32 of the result's shape")
@@ -192,7 +202,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
                 ptr(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages),
                 0 if k_pages is None else k_pages.shape[0], ptr(block_table), table_width, ring_pages, page_tokens,
                 ptr(cu_seqlens), ptr(start_pos), n_seqs, T, int(window or 0), float(scale), float(softcap or 0.0),
-                ptr(slopes), keep, int(sink), g_ptr, g_ld, ptr(out), n_heads, n_kv_heads, key_dim,
+                ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, ptr(out), n_heads, n_kv_heads, key_dim,
                 ptr(tc_status_word(q.device)), stream())
             if st != NOT_SUPPORTED:
                 check(st, "flash_prefill_tc_ext")
@@ -200,7 +210,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
             st = core().tq_flash_prefill_ext(
                 ptr(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages), ptr(block_table), table_width,
                 ring_pages, page_tokens, ptr(cu_seqlens), ptr(start_pos), n_seqs, T, int(window or 0), float(scale),
-                float(softcap or 0.0), ptr(slopes), keep, int(sink), g_ptr, g_ld, ptr(out), n_heads, n_kv_heads,
+                float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, ptr(out), n_heads, n_kv_heads,
                 key_dim, stream())
             if st != NOT_SUPPORTED:
                 check(st, "flash_prefill_ext")
@@ -212,13 +222,14 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
     if fast and not packed:
         st = core().tq_flash_decode_ext(
             ptr(q), ptr(k_pages), ptr(v_pages), ptr(block_table), table_width, ring_pages, page_tokens, ptr(tok_pos),
-            ptr(tok_seq), int(window or 0), float(scale), float(softcap or 0.0), ptr(slopes), keep, int(sink),
+            ptr(tok_seq), int(window or 0), float(scale), float(softcap or 0.0), ptr(slopes), keep, ptr(sink),
+            int(chunk or 0),
             ptr(out), ptr(part_acc), ptr(part_ml), T, n_heads, n_kv_heads, key_dim, n_splits, stream())
         if st != NOT_SUPPORTED:
             check(st, "flash_decode_ext")
             if n_splits > 1:
                 check(core().tq_attention_merge(ptr(part_acc), ptr(part_ml), ptr(out), dtype_code(out), T, n_heads,
-                                                value_dim, n_splits, int(sink), stream()), "attention_merge")
+                                                value_dim, n_splits, ptr(sink), stream()), "attention_merge")
             if gate is not None:
                 from .elementwise import sigmoid_gate
                 sigmoid_gate(out, gate)
@@ -227,7 +238,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
         ptr(q), dtype_code(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages), ptr(block_table),
         table_width, ring_pages, page_tokens, ptr(tok_pos), ptr(tok_seq), ptr(cu_seqlens), ptr(start_pos),
         int(window or 0), float(scale), ptr(out), ptr(part_acc), ptr(part_ml), T, n_heads, n_kv_heads, key_dim,
-        value_dim, float(softcap or 0.0), ptr(slopes), keep, int(sink), n_splits, stream()),
+        value_dim, float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), n_splits, stream()),
         "attention_ext", 2 if n_splits > 1 else 1)
     if gate is not None:
         from .elementwise import sigmoid_gate

@@ -71,13 +71,23 @@ def qkv_rope_cache(qkv, bias, cos, sin, tok_pos, tok_seq, new_lens, q_out, *, n_
 
 
 ACT_SILU, ACT_GELU_TANH = 1, 2          # the gate's activation in a gated feed-forward (csrc/common.cuh)
+ACT_SQUARE_RELU = 3                     # of plain products only (kernels.linear)
 
 
 def activation_code(name: str) -> int:
     try:
-        return {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH}[name]
+        return {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "square_relu": ACT_SQUARE_RELU}[name]
     except KeyError:
         raise KernelError(f"unknown gate activation '{name}' (silu, gelu_tanh)") from None
+
+
+def square_relu(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = max(x, 0)^2: float32 rows x (may be `out` itself) into contiguous out [T, n]."""
+    if x.dtype != torch.float32 or x.stride(1) != 1 or out.shape != x.shape:
+        raise KernelError("square_relu: x float32 [T, n], out of its shape")
+    need_contiguous(out=out)
+    check(core().tq_square_relu(ptr(x), x.stride(0), ptr(out), dtype_code(out), x.shape[0], x.shape[1], stream()), "square_relu")
+    return out
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU):
@@ -225,14 +235,16 @@ def head_encode(proj: torch.Tensor, ctx_pos, q_out: torch.Tensor, *, q_col: int,
                 n_heads: int, n_kv_heads: int, key_dim: int, value_dim: int, cos=None, sin=None, rotary_dim: int = 0,
                 norm_eps: float = 0.0, k_out=None, v_out=None, k_pages=None, v_pages=None, block_table=None,
                 table_width: int = 0, ring_pages: int = 0, page_tokens: int = 64, paired: bool = False,
-                row_inv=None, q_weight=None, k_weight=None):
+                row_inv=None, q_weight=None, k_weight=None, v_scale: float = 1.0):
     """From projected float32 rows [T, ld] (q heads from column q_col, k heads from k_col, v heads from v_col; with
     v_col < 0 the values are the keys as projected) to encoded q, and k / v packed and / or appended to the cache
     (see csrc/head_encode.cu).  `ctx_pos` = (tok_pos, tok_seq, new_lens).  q and k are rotated over their first
     `rotary_dim` entries (cos/sin float32 [positions, rotary_dim/2]; entry i with i + rotary_dim/2, or with
     `paired` entry 2i with 2i + 1) or, with norm_eps > 0, divided by their root mean square per head.  With
     `row_inv` (float32 [T, 2] from `row_inv_rms`) and the weights q_weight [n_heads * key_dim] and k_weight
-    [n_kv_heads * key_dim], q and k are first normed over their whole rows.  n_kv_heads may be 0: only q is encoded."""
+    [n_kv_heads * key_dim], q and k are first normed over their whole rows; with norm_eps and weights [key_dim] (shared
+    by the heads) each head is normed and weighted before it is rotated.  The values leave times `v_scale`.
+    n_kv_heads may be 0: only q is encoded."""
     tok_pos, tok_seq, new_lens = ctx_pos
     T, ld = proj.shape
     if proj.dtype != torch.float32 or proj.stride(1) != 1:
@@ -256,13 +268,18 @@ def head_encode(proj: torch.Tensor, ctx_pos, q_out: torch.Tensor, *, q_col: int,
                                     or k_weight.shape[0] != n_kv_heads * key_dim))):
             raise KernelError("head_encode: row_inv float32 [T, 2] needs float32 weights over the whole q and k rows")
         need_contiguous(row_inv=row_inv, q_weight=q_weight, k_weight=k_weight)
+    elif q_weight is not None or k_weight is not None:
+        for w in (q_weight, k_weight):
+            if not norm_eps > 0.0 or w is None or w.dtype != torch.float32 or tuple(w.shape) != (key_dim,):
+                raise KernelError("head_encode: a norm per head takes norm_eps and float32 weights [key_dim] for q and k")
+        need_contiguous(q_weight=q_weight, k_weight=k_weight)
     need_contiguous(q_out=q_out, k_out=k_out, v_out=v_out, k_pages=k_pages, v_pages=v_pages, block_table=block_table,
                     cos=cos, sin=sin)
     check(core().tq_head_encode(ptr(proj), proj.stride(0), q_col, k_col, v_col, ptr(cos), ptr(sin), rotary_dim,
                                 float(norm_eps), ptr(tok_pos), ptr(tok_seq), ptr(new_lens), ptr(block_table),
                                 table_width, ring_pages, page_tokens, ptr(q_out), ptr(k_out), ptr(v_out), ptr(k_pages),
                                 ptr(v_pages), dtype_code(q_out), T, n_heads, n_kv_heads, key_dim, value_dim,
-                                ptr(row_inv), ptr(q_weight), ptr(k_weight), int(bool(paired)), stream()),
+                                ptr(row_inv), ptr(q_weight), ptr(k_weight), int(bool(paired)), float(v_scale), stream()),
           "head_encode")
     return q_out
 

@@ -95,8 +95,9 @@ def _tc_takes(rows: int, w: torch.Tensor, swiglu: bool, after_norm: bool, float3
 
 
 def _gate(swiglu, activation) -> int:
-    """The `swiglu` argument of the C functions: 0 for a plain product, else the gate's activation code."""
-    return int(activation) if swiglu else 0
+    """The `swiglu` argument of the C functions: 0 for a plain product, ACT_SQUARE_RELU for a plain one with that
+    activation on its result, else the gate's activation code."""
+    return int(activation) if swiglu or activation == elementwise.ACT_SQUARE_RELU else 0
 
 
 def skinny_gemm(x, w, out, bias=None, accumulate=False, swiglu=False, activation=elementwise.ACT_SILU):
@@ -112,7 +113,7 @@ def skinny_gemm(x, w, out, bias=None, accumulate=False, swiglu=False, activation
 
 # ---- tcgen05 + TMA product for many rows (csrc/gemm_tc.cu) -----------------------
 USE_TCGEN05 = True                  # False: the library product (cuBLAS) takes the many-row bfloat16 case
-EPI_STORE, EPI_ACCUM, EPI_SWIGLU, EPI_GELU = 0, 1, 2, 3
+EPI_STORE, EPI_ACCUM, EPI_SWIGLU, EPI_GELU, EPI_RELU2 = 0, 1, 2, 3, 4
 
 
 def set_gemm_tc_mode(mode: int) -> None:
@@ -217,8 +218,7 @@ def gemv_rows(x, w, out, bias=None, accumulate=False, swiglu=False, activation=e
     N = out.shape[1]
     check(core().tq_gemv_rows(ptr(x), dtype_code(x), ptr(w), dtype_code(w), ptr(bias), ptr(out), dtype_code(out),
                               M, N, K, x.stride(0), w.stride(0), out.stride(0), int(accumulate),
-                              int(activation) if swiglu else 0,
-                              stream()), "gemv_rows")
+                              _gate(swiglu, activation), stream()), "gemv_rows")
     return out
 
 
@@ -226,10 +226,14 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = N
            out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
            accumulate: bool = False, swiglu: bool = False, activation: int = elementwise.ACT_SILU) -> torch.Tensor:
     """y = x · w^T (+ bias); with `swiglu`, w holds gate rows then up rows and
-    y = act(x · gate^T) * (x · up^T), act being silu unless `activation` names another; with `accumulate`, `out` (float32) gets
+    y = act(x · gate^T) * (x · up^T), act being silu unless `activation` names another; without it and with
+    `activation` ACT_SQUARE_RELU, y = max(x · w^T + bias, 0)^2 (not with `accumulate`); with `accumulate`, `out` (float32) gets
     y added to it.  x [M, K], w [N, K] (or [2N, K]); float32 accumulation
     throughout."""
     pending = x if isinstance(x, PendingNorm) else None
+    relu2 = activation == elementwise.ACT_SQUARE_RELU
+    if relu2 and (swiglu or accumulate):
+        raise KernelError("linear: the square of relu is an activation of plain products that are not accumulated")
     if len(x.shape) != 2 or w.dim() != 2 or x.shape[1] != w.shape[1]:
         raise KernelError(f"linear: shapes {tuple(x.shape)} and {tuple(w.shape)} do not multiply")
     if (pending is None and x.stride(1) != 1) or w.stride(1) != 1:
@@ -251,13 +255,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = N
     if M == 0:
         return out
     if pending is not None:
-        if _fused_norm(pending, w, out, bias, accumulate, swiglu, activation):
+        if not relu2 and _fused_norm(pending, w, out, bias, accumulate, swiglu, activation):
             return out
         x = pending.materialize()
 
     # decoding: the TMA-fed tcgen05 kernel or the mma.sync kernel (_tc_takes says which, where both can)
     if (USE_TCGEN05 and M <= SKINNY_MAX_ROWS and _tc_ok(x, w, out, swiglu)
-            and (not accumulate or out.dtype == torch.float32)
+            and (not accumulate or out.dtype == torch.float32) and not (relu2 and out.dtype != torch.bfloat16)
             and (not _skinny_ok(x, w)
                  or _tc_takes(M, w, bool(swiglu), pending is not None, out.dtype == torch.float32))):
         return decode_gemm_tc(x, w, out, bias, accumulate, swiglu, activation)
@@ -266,14 +270,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = N
     if M <= ROW_KERNEL_MAX_ROWS:
         return gemv_rows(x, w, out, bias, accumulate, swiglu, activation)
 
-    if _tc_ok(x, w, out, swiglu) and (not accumulate or out.dtype == torch.float32):
+    if (_tc_ok(x, w, out, swiglu) and (not accumulate or out.dtype == torch.float32)
+            and not (relu2 and out.dtype != torch.bfloat16)):
         gated = EPI_GELU if activation == elementwise.ACT_GELU_TANH else EPI_SWIGLU
-        return gemm_tc(x, w, out, bias, gated if swiglu else (EPI_ACCUM if accumulate else EPI_STORE))
+        plain = EPI_RELU2 if relu2 else (EPI_ACCUM if accumulate else EPI_STORE)
+        return gemm_tc(x, w, out, bias, gated if swiglu else plain)
 
     if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and bias is None:
         y = torch.mm(x, w.t(), out_dtype=torch.float32)          # library product, float32 out
         if swiglu:
             return elementwise.swiglu(y, out, activation)
+        if relu2:
+            return elementwise.square_relu(y, out)
         if accumulate:
             return elementwise.add_into(out, y)
         if out.dtype == torch.float32:
@@ -286,4 +294,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = N
         y = torch.empty((M, rows_w), dtype=torch.float32, device=x.device)
         gemm_tiled(x, w, y, bias, False)
         return elementwise.swiglu(y, out, activation)
+    if relu2:
+        y = out if out.dtype == torch.float32 and out.is_contiguous() else torch.empty((M, N), dtype=torch.float32, device=x.device)
+        gemm_tiled(x, w, y, bias, False)
+        return elementwise.square_relu(y, out)
     return gemm_tiled(x, w, out, bias, accumulate)

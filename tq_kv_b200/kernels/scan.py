@@ -89,7 +89,7 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
     `regions`: (first channel, channels, vector width, unit, scale) — each vector of a region with `unit` leaves
     as x * scale / sqrt(sum(x^2) + unit_eps).  With `gate_raw` float32 [T, H] the per-token scalars of a
     recurrence go to `scalars` float32 [T, H, 4]: g = exp(-exp(a_log) * softplus(gate_raw + dt_bias)), then
-    sigmoid(beta_raw) if given, else the softplus itself."""
+    sigmoid(beta_raw) if given, else the softplus itself; with `beta_raw` alone they are (1, sigmoid(beta_raw))."""
     T, C = x.shape
     K = weight.shape[1]
     if x.dtype != torch.float32 or out.dtype != torch.float32 or state.dtype != torch.float32 or weight.dtype != torch.float32:
@@ -130,6 +130,13 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
                 raise KernelError("short_conv: beta_raw must be float32 [T, H]")
             ldb = beta_raw.stride(0)
         need_contiguous(a_log=a_log, dt_bias=dt_bias, scalars=scalars)
+    elif beta_raw is not None:
+        H = beta_raw.shape[1]
+        if (beta_raw.dtype != torch.float32 or beta_raw.shape[0] != T or beta_raw.stride(1) != 1 or scalars is None
+                or scalars.dtype != torch.float32 or tuple(scalars.shape) != (T, H, 4)):
+            raise KernelError("short_conv: beta_raw float32 [T, H] needs scalars float32 [T, H, 4]")
+        ldb = beta_raw.stride(0)
+        need_contiguous(scalars=scalars)
     need_contiguous(weight=weight, bias=bias, tok_seq=tok_seq, cu_seqlens=cu_seqlens, slots=slots)
     n_kernels = 1 if single_tokens or K == 1 else 2
     check(core().tq_short_conv(ptr(x), x.stride(0), ptr(weight), ptr(bias), ptr(out), out.stride(0), ptr(state),
@@ -172,4 +179,36 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scalars: torch
     check(core().tq_gated_scan(int(bool(delta)), ptr(q), ptr(k), ptr(v), q.stride(0), ptr(scalars), ptr(skip),
                                heads // qk_heads, ptr(state), state.stride(0), ptr(cu_seqlens), ptr(slots), int(n_seqs),
                                T, int(single_tokens), ptr(out), out.stride(0), heads, d, e, stream()), "gated_scan")
+    return out
+
+
+def channel_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor,
+                       state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, out: torch.Tensor, *,
+                       n_seqs: int, heads: int, qk_heads: int, key_dim: int, value_dim: int, single_tokens: bool = False):
+    """The delta rule with a decay per head and key channel:  S' = diag(w) S;  S = S' + k (beta (v - S'^T k))^T;
+    o = S^T q.  Operands as in `gated_scan`; `decay` float32 [T, heads * d] holds w, of `scalars` only beta (entry 1)
+    is read."""
+    T = q.shape[0]
+    d, e = int(key_dim), int(value_dim)
+    for name, t, n in (("q", q, qk_heads * d), ("k", k, qk_heads * d), ("v", v, heads * e)):
+        if t.dtype != torch.float32 or tuple(t.shape) != (T, n) or t.stride(1) != 1 or t.stride(0) != q.stride(0):
+            raise KernelError(f"channel_delta_scan: {name} must be float32 [T, {n}], a column slice of the buffer q lies in")
+    if heads % qk_heads or not 0 < d <= MAX_KEY_WIDTH:
+        raise KernelError(f"channel_delta_scan: {heads} heads cannot share {qk_heads} key heads, or key width {d} is "
+                          f"outside 1..{MAX_KEY_WIDTH}")
+    if decay.dtype != torch.float32 or tuple(decay.shape) != (T, heads * d) or decay.stride(1) != 1:
+        raise KernelError("channel_delta_scan: decay must be float32 [T, heads * d]")
+    if scalars.dtype != torch.float32 or tuple(scalars.shape) != (T, heads, 4) or not scalars.is_contiguous():
+        raise KernelError("channel_delta_scan: scalars must be float32 [T, heads, 4]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < heads * d * e:
+        raise KernelError("channel_delta_scan: state must be float32 [slots, >= heads * d * e]")
+    if out.dtype != torch.float32 or tuple(out.shape) != (T, heads * e) or out.stride(1) != 1:
+        raise KernelError("channel_delta_scan: out must be float32 [T, heads * e]")
+    if single_tokens and T != n_seqs:
+        raise KernelError("channel_delta_scan: single_tokens needs one token per sequence")
+    need_contiguous(cu_seqlens=cu_seqlens, slots=slots)
+    check(core().tq_channel_delta_scan(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(decay), decay.stride(0), ptr(scalars),
+                                       heads // qk_heads, ptr(state), state.stride(0), ptr(cu_seqlens), ptr(slots),
+                                       int(n_seqs), T, int(single_tokens), ptr(out), out.stride(0), heads, d, e, stream()),
+          "channel_delta_scan")
     return out

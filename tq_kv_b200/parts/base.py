@@ -109,6 +109,7 @@ class StepContext:
     # that lives for one step: an entry that brings a prompt's keys and values along as packed rows may leave them
     # there for the entries that read its cache, which then need not find them in pages.
     cache_entry: int = -1
+    rider_out: Optional[torch.Tensor] = None    # see Part.accepts_rider
     step_shared: Optional[dict] = None
 
 
@@ -129,6 +130,11 @@ class Part:
     takes_pending_norm = False
     # A mixer or feed-forward that honours StepContext.store_result (see there).
     can_store_result = False
+    # A mixer or feed-forward whose first product can carry another part's rows: where the block sets `rider` (a part
+    # with `rider_rows()`, bound earlier), its weight rows ride in that product and their float32 results are left in
+    # StepContext.rider_out, so that what reads the same input costs no product of its own.
+    accepts_rider = False
+    rider: Optional["Part"] = None
 
     def __init__(self, spec: PartSpec):
         self.spec = spec
@@ -190,3 +196,25 @@ def shapes_agree(want, got) -> bool:
 
 def float32_vector(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float32).contiguous()
+
+
+def stack_rows(weights: list[torch.Tensor], biases: Optional[list[Optional[torch.Tensor]]] = None,
+               multiple: int = 8) -> tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """The weights' rows one below the other, for one product, filled up with zero rows to a multiple of `multiple`
+    (the tensor-core kernels hand out results in 16-byte pieces), and the float32 bias over all rows (None if no
+    weight has one).  Weights of different dtypes are widened to float32."""
+    if len({w.dtype for w in weights}) != 1:
+        weights = [w.to(torch.float32) for w in weights]
+    n = sum(w.shape[0] for w in weights)
+    pad = -n % multiple
+    if pad:
+        weights = [*weights, weights[0].new_zeros((pad, weights[0].shape[1]))]
+    bias = None
+    if biases is not None and any(b is not None for b in biases):
+        bias = torch.zeros(n + pad, dtype=torch.float32, device=weights[0].device)
+        at = 0
+        for w, b in zip(weights, biases):
+            if b is not None:
+                bias[at:at + w.shape[0]] = b
+            at += w.shape[0]
+    return torch.cat(weights, dim=0).contiguous(), bias

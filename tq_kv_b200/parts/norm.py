@@ -33,6 +33,10 @@ class RMSNorm(Norm):
         if self.weight_offset != 0.0:
             self.weight = (self.weight + self.weight_offset).contiguous()
 
+    def stream_args(self) -> dict:
+        """The norm as arguments of `kernels.streams_step`, which can apply it to what it reads."""
+        return {"norm_weight": self.weight, "eps": self.eps}
+
     def forward(self, x, out_dtype, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.width), dtype=out_dtype, device=x.device)
@@ -56,8 +60,39 @@ class GroupRMSNorm(RMSNorm):
             raise ConfigError(f"a norm over {self.width} values cannot be cut into {self.groups} equal groups")
         if self.groups > 1:
             self.pending = None             # the products fold in the plain norm only
+            self.stream_args = None         # ... and so do the residual streams' kernels
 
     def forward(self, x, out_dtype, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.width), dtype=out_dtype, device=x.device)
         return kernels.group_rmsnorm(x, self.weight, self.eps, out, groups=self.groups, rows=rows)
+
+
+class DynamicTanhNorm(Norm):
+    """A norm without statistics: tanh(alpha * x) * weight + bias, entry by entry in float32; alpha is one learned
+    number (tensor `<weight_name>.alpha`), weight and bias (`<weight_name>.b`) have the row's width."""
+    padded_rows_ok = True
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.width = int(self.params["width"])
+        self.weight_name = self.params.get("weight_name") or self.prefix + "weight"
+        self.weight = self.bias = self.alpha = self._one = None
+
+    def weight_specs(self):
+        n = self.weight_name
+        return [WeightSpec(n, (self.width,), "norm_scale"), WeightSpec(n + ".b", (self.width,), "bias"),
+                WeightSpec(n + ".alpha", (), "tanh_alpha")]
+
+    def bind(self, tensors, runtime: Runtime, shared=None):
+        n = self.weight_name
+        self.weight, self.bias = float32_vector(tensors[n]), float32_vector(tensors[n + ".b"])
+        self.alpha = float32_vector(tensors[n + ".alpha"].reshape(1))
+        self._one = torch.ones(1, dtype=torch.float32, device=self.weight.device)
+
+    def stream_args(self) -> dict:
+        return {"norm_weight": self.weight, "norm_bias": self.bias, "alpha": self.alpha}
+
+    def forward(self, x, out_dtype, rows=None):
+        # one stream that is read and not written (csrc/stream_mix.cu)
+        return kernels.streams_step(x.unsqueeze(0), read=self._one, out_dtype=out_dtype, rows=rows, **self.stream_args())

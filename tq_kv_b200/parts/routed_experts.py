@@ -1,6 +1,7 @@
-"""A feed-forward of `experts` small SwiGLU layers of which each token uses `top`.
+"""A feed-forward of `experts` small layers of which each token uses `top`.
 
-Expert e is  W_down[e] (silu(W_gate[e] x) * (W_up[e] x)),  no biases.  Which experts a
+Expert e is  W_down[e] (silu(W_gate[e] x) * (W_up[e] x)),  or with `gated` False
+W_down[e] max(W_up[e] x, 0)^2;  no biases.  Which experts a
 token uses is `routing`:
   "table"   there is no router: a table [vocab, top] of expert indices (the
             entries of a row differ) names them by the token's id; each has the
@@ -8,6 +9,11 @@ token uses is `routing`:
   "router"  scores s = sigmoid(W_router x), computed in float32; the `top` experts
             with the largest scores are chosen (the lowest index first among equals);
             their weights are  router_scale * s / (sum of the chosen s + weight_sum_floor).
+  "group_router"  scores s = softmax(W_router x) over all experts, in float32; the choice
+            goes by s + correction (a learned number per expert): the experts lie in
+            `groups` equal groups of neighbours, a group counts as its largest choice
+            score, and of the `keep_groups` best groups' experts the `top` best are
+            chosen; their weights are their s as they are.
 The result is the weighted sum of the chosen experts' results.  With `shared_size` > 0
 a shared expert of that inner width (same form, tensors under `names["shared"]`) runs
 for every token and is added.
@@ -25,7 +31,7 @@ import torch
 
 from .. import kernels
 from ..config import ConfigError
-from .base import FeedForward, Runtime, StepContext, WeightSpec
+from .base import FeedForward, Runtime, StepContext, WeightSpec, float32_vector, stack_rows
 
 
 class TableExperts(FeedForward):
@@ -45,8 +51,17 @@ class TableExperts(FeedForward):
         self.n_experts = int(p["experts"])
         self.top = int(p["top"])
         self.routing = p.get("routing", "table")
-        if self.routing not in ("table", "router"):
-            raise ConfigError(f"routed experts: unknown routing '{self.routing}' (known: table, router)")
+        if self.routing not in ("table", "router", "group_router"):
+            raise ConfigError(f"routed experts: unknown routing '{self.routing}' (known: table, router, group_router)")
+        self.gated = bool(p.get("gated", True))
+        self.groups, self.keep_groups = int(p.get("groups", 1)), int(p.get("keep_groups", 1))
+        if self.routing == "group_router":
+            if self.groups < 1 or self.n_experts % self.groups or not 1 <= self.keep_groups <= self.groups:
+                raise ConfigError(f"routed experts: {self.n_experts} experts in {self.groups} equal groups, {self.keep_groups} kept")
+            if self.top > self.keep_groups * (self.n_experts // self.groups):
+                raise ConfigError(f"routed experts: a token cannot use {self.top} experts of {self.keep_groups} groups of "
+                                  f"{self.n_experts // self.groups}")
+        self.accepts_rider = self.routing == "group_router"      # (rows beside the router's)
         self.vocab = int(p["vocab_size"]) if self.routing == "table" else 0
         self.router_scale = float(p.get("router_scale", 1.0))
         self.weight_sum_floor = float(p.get("weight_sum_floor", 0.0))
@@ -56,7 +71,10 @@ class TableExperts(FeedForward):
         self.names = dict(p.get("names", {"expert": "e{}.", "gate": "gate", "up": "up", "down": "down", "table": "table"}))
         self.names.setdefault("router", "router")
         self.names.setdefault("shared", "shared.")
+        self.names.setdefault("correction", "correction")
         self.w_gate_up = self.w_down = self.table = self.w_router = self.w_shared_gate_up = self.w_shared_down = None
+        self.correction = self.router_bias = None
+        self.projections = ("gate", "up") if self.gated else ("up",)      # the rows of an expert's first product
 
     def _e(self, e: int, which: str) -> str:
         return f"{self.prefix}{self.names['expert'].format(e)}{self.names[which]}"
@@ -64,37 +82,45 @@ class TableExperts(FeedForward):
     def weight_specs(self):
         specs = []
         for e in range(self.n_experts):
-            specs += [WeightSpec(self._e(e, "gate"), (self.inter, self.hidden), "matrix"),
-                      WeightSpec(self._e(e, "up"), (self.inter, self.hidden), "matrix"),
-                      WeightSpec(self._e(e, "down"), (self.hidden, self.inter), "matrix")]
+            specs += [WeightSpec(self._e(e, w), (self.inter, self.hidden), "matrix") for w in self.projections]
+            specs.append(WeightSpec(self._e(e, "down"), (self.hidden, self.inter), "matrix"))
         if self.routing == "table":
             specs.append(WeightSpec(self.prefix + self.names["table"], (self.vocab, self.top),
                                     f"choice_table:{self.n_experts}"))
         else:
             specs.append(WeightSpec(self.prefix + self.names["router"], (self.n_experts, self.hidden), "matrix"))
+        if self.routing == "group_router":
+            specs.append(WeightSpec(self.prefix + self.names["correction"], (self.n_experts,), "bias"))
         if self.shared_size:
             sp = self.prefix + self.names["shared"]
-            specs += [WeightSpec(sp + self.names["gate"], (self.shared_size, self.hidden), "matrix"),
-                      WeightSpec(sp + self.names["up"], (self.shared_size, self.hidden), "matrix"),
-                      WeightSpec(sp + self.names["down"], (self.hidden, self.shared_size), "matrix")]
+            specs += [WeightSpec(sp + self.names[w], (self.shared_size, self.hidden), "matrix") for w in self.projections]
+            specs.append(WeightSpec(sp + self.names["down"], (self.hidden, self.shared_size), "matrix"))
         return specs
 
     def bind(self, tensors, runtime: Runtime, shared=None):
-        mats = [tensors[self._e(e, w)] for e in range(self.n_experts) for w in ("gate", "up", "down")]
+        n = len(self.projections)
+        mats = [tensors[self._e(e, w)] for e in range(self.n_experts) for w in (*self.projections, "down")]
         if len({m.dtype for m in mats}) != 1:
             mats = [m.to(torch.float32) for m in mats]
-        gu = [torch.cat([mats[3 * e], mats[3 * e + 1]], dim=0) for e in range(self.n_experts)]
-        self.w_gate_up = torch.stack(gu).contiguous()                                       # [E, 2F, W]
-        self.w_down = torch.stack([mats[3 * e + 2] for e in range(self.n_experts)]).contiguous()   # [E, W, F]
+        gu = [torch.cat(mats[(n + 1) * e:(n + 1) * e + n], dim=0) for e in range(self.n_experts)]
+        self.w_gate_up = torch.stack(gu).contiguous()                        # [E, 2F, W] (without a gate [E, F, W])
+        self.w_down = torch.stack([mats[(n + 1) * e + n] for e in range(self.n_experts)]).contiguous()   # [E, W, F]
         if self.shared_size:
             sp = self.prefix + self.names["shared"]
-            g, u = tensors[sp + self.names["gate"]], tensors[sp + self.names["up"]]
-            if g.dtype != u.dtype:
-                g, u = g.to(torch.float32), u.to(torch.float32)
-            self.w_shared_gate_up = torch.cat([g, u], dim=0).contiguous()
+            rows = [tensors[sp + self.names[w]] for w in self.projections]
+            if len({r.dtype for r in rows}) != 1:
+                rows = [r.to(torch.float32) for r in rows]
+            self.w_shared_gate_up = torch.cat(rows, dim=0).contiguous()
             self.w_shared_down = tensors[sp + self.names["down"]].contiguous()
         if self.routing == "router":
             self.w_router = tensors[self.prefix + self.names["router"]].contiguous()
+            return
+        if self.routing == "group_router":           # the rider's rows first: their columns then start aligned
+            rows = ([self.rider.rider_rows()] if self.rider is not None else []) \
+                + [(tensors[self.prefix + self.names["router"]], None)]
+            self.w_router, self.router_bias = stack_rows([w for w, _ in rows], [b for _, b in rows])
+            self.router_col = rows[0][0].shape[0] if self.rider is not None else 0
+            self.correction = float32_vector(tensors[self.prefix + self.names["correction"]])
             return
         table = tensors[self.prefix + self.names["table"]]
         if table.dtype != torch.int32:
@@ -108,19 +134,27 @@ class TableExperts(FeedForward):
         weights = None
         if self.routing == "table":
             choice = kernels.table_choice(ctx.batch.tokens, self.table, self.n_experts)
+        elif self.routing == "group_router":
+            proj = kernels.linear(x, self.w_router, bias=self.router_bias, out_dtype=torch.float32)
+            kernels.mark("router")
+            if self.rider is not None:
+                ctx.rider_out = proj[:, :self.router_col]
+            choice, weights = kernels.group_router_choice(proj[:, self.router_col:self.router_col + self.n_experts],
+                                                          self.top, self.correction, self.groups, self.keep_groups)
         else:
             logits = kernels.linear(x, self.w_router, out_dtype=torch.float32)
             choice, weights = kernels.router_choice(logits, self.top, self.router_scale, self.weight_sum_floor)
         T = x.shape[0]
         if ((T >= self.TILE_MIN_ROWS or T * self.top >= self.TILE_MIN_PAIRS_PER_EXPERT * self.n_experts)
-                and x.dtype == torch.bfloat16 and kernels.routed_tiles_ok(x, self.w_gate_up, self.w_down)):
+                and x.dtype == torch.bfloat16 and kernels.routed_tiles_ok(x, self.w_gate_up, self.w_down, self.gated)):
             kernels.routed_experts_tiles(x, self.w_gate_up, self.w_down, choice, residual,
-                                         accumulate=not ctx.store_result, weights=weights)
+                                         accumulate=not ctx.store_result, weights=weights, gated=self.gated)
         else:
             kernels.routed_experts_rows(x, self.w_gate_up, self.w_down, choice, residual,
-                                        accumulate=not ctx.store_result, weights=weights)
+                                        accumulate=not ctx.store_result, weights=weights, gated=self.gated)
         kernels.mark("experts")
         if self.shared_size:
-            act = kernels.linear(x, self.w_shared_gate_up, swiglu=True, out_dtype=ctx.runtime.act_dtype)
+            act = kernels.linear(x, self.w_shared_gate_up, swiglu=self.gated, out_dtype=ctx.runtime.act_dtype,
+                                 activation=kernels.ACT_SILU if self.gated else kernels.ACT_SQUARE_RELU)
             kernels.linear(act, self.w_shared_down, out=residual, accumulate=True)
             kernels.mark("shared_expert")

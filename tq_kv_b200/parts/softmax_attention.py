@@ -8,8 +8,9 @@
   row_norm_eps      q and k are RMS-normed over their WHOLE projections (all heads of a
                     token at once, x / sqrt(mean(x^2) + eps) * weight, weights `q_norm` and
                     `k_norm` of the projections' sizes) before the heads are split and rotated
-  sink              the softmax's denominator counts one more key of score 0 that has no
-                    value: p_j = exp(s_j) / (1 + sum exp(s))
+  sink              the softmax's denominator counts one more key that has no value, of score
+                    0 (True), p_j = exp(s_j) / (1 + sum exp(s)), or ("learned") of a score per
+                    head, the tensor `sink` [heads]: p_j = exp(s_j) / (exp(sink_h) + sum exp(s))
   shared_kv         the layer has no key/value tensors: it reads the cache of the schedule
                     entry it is given (whose keys are stored normed and rotated) with its own
                     queries, window and everything else
@@ -18,16 +19,21 @@
   shares_packed     a prompt's packed keys and values are left in the step's shared dict for
                     the layers that read this layer's cache
   qk_norm_eps       q and k are divided per head by their root mean square,
-                    x / sqrt(mean(x^2) + eps), without a weight
+                    x / sqrt(mean(x^2) + eps), without a weight, or with `qk_norm_weights` times
+                    the weights `q_norm` and `k_norm` [d], which the heads share; then rotated
   scale             s = q . k * scale
   softcap           s <- softcap * tanh(s / softcap)
   slope_exponent    a bias that grows with the distance: s <- s - m_h * (i - j),
                     m_h = 2^(-slope_exponent * (h + 1) / heads) for head h = 0 ..
   window            the query at position i sees key j <= i if i - j < window
+  chunk             (instead of a window) the query at position i sees key j <= i if
+                    i // chunk == j // chunk; chunks are counted from position 0
   keep_first        ... or if j < keep_first (the first tokens stay visible; they keep
                     their true positions)
   output_gate       the heads side by side are multiplied entry by entry with
                     sigmoid(W_g x) before the output projection
+  result_scale      the mixer's result is multiplied by it: the values are, before they are
+                    rounded and cached (the result is linear in them)
 Query head h reads key/value head h // (heads / kv_heads).  Key rows and value rows
 may differ in width; widths that are no multiple of 8 are padded with zeros inside.
 No biases.
@@ -35,7 +41,7 @@ No biases.
 All projections are one product with the concatenated weight (float32 result); one
 kernel encodes q and k, splits the heads and appends k and v to the cache
 (csrc/head_encode.cu).  Prompts from position 0 attend over the step's own keys;
-everything else reads the paged cache: a ring for a plain window, all keys where
+everything else reads the paged cache: a ring for a plain window or chunks, all keys where
 first tokens are kept (the kernels skip what lies between the kept tokens and the
 window).  Scores, softmax and the bias are float32.  bfloat16 steps whose keys and
 values have one width run the tensor-core kernels (`kernels.attention_ext`), which
@@ -90,15 +96,27 @@ class SoftmaxAttention(Mixer):
             self.qk_norm_eps *= ratio
             self.scale *= ratio
         self.window: Optional[int] = int(p["window"]) if p.get("window") else None
-        self.cache_window: Optional[int] = self.window
+        self.chunk: Optional[int] = int(p["chunk"]) if p.get("chunk") else None
+        if self.window and self.chunk:
+            raise ConfigError("softmax attention: a window or chunks, not both")
+        self.span = self.window or self.chunk                # the most keys a query sees (None: all)
+        self.cache_window: Optional[int] = self.span
         if "cache_window" in p:
             self.cache_window = int(p["cache_window"]) if p.get("cache_window") else None
-        if self.window is None and self.cache_window is not None:
+        if self.span is None and self.cache_window is not None:
             raise ConfigError("softmax attention: a layer without a window needs a cache of all keys")
-        if self.window is not None and self.cache_window is not None and self.cache_window < self.window:
-            raise ConfigError(f"softmax attention: a cache of {self.cache_window} keys is too small for a window of {self.window}")
+        if self.span is not None and self.cache_window is not None and self.cache_window < self.span:
+            raise ConfigError(f"softmax attention: a cache of {self.cache_window} keys is too small for a window of {self.span}")
         self.row_norm_eps = float(p["row_norm_eps"]) if p.get("row_norm_eps") else 0.0
-        self.sink = bool(p.get("sink", False))
+        self.sink = p.get("sink", False)
+        if self.sink not in (False, True, "learned"):
+            raise ConfigError(f"softmax attention: sink '{self.sink}' (False, True or learned)")
+        self.qk_norm_weights = bool(p.get("qk_norm_weights", False))
+        if self.qk_norm_weights and not self.qk_norm_eps:
+            raise ConfigError("softmax attention: qk_norm_weights belong to a norm per head (qk_norm_eps)")
+        self.result_scale = float(p.get("result_scale", 1.0))
+        if self.result_scale != 1.0 and self.shared_kv_given(p):
+            raise ConfigError("softmax attention: result_scale rides in the values, a layer that reads another's cache has none")
         self.shared_kv = bool(p.get("shared_kv", False))
         self.shares_packed = bool(p.get("shares_packed", False))
         if self.shared_kv and self.values != "projected":
@@ -114,16 +132,18 @@ class SoftmaxAttention(Mixer):
             if self.position.rotary_dim > self.key_dim_given:
                 raise ConfigError(f"softmax attention: {self.position.rotary_dim} rotated entries in heads of "
                                   f"{self.key_dim_given}")
-            if self.qk_norm_eps:
-                raise ConfigError("softmax attention: either a rotation or unit-size q and k, not both")
         if self.qk_norm_eps and self.row_norm_eps:
             raise ConfigError("softmax attention: q and k are normed per head or over the whole row, not both")
         self.q_width = self.n_heads * self.key_dim
         self.k_width = 0 if self.shared_kv else self.n_kv_heads * self.key_dim
         self.v_width = self.n_kv_heads * self.value_dim if self.values == "projected" and not self.shared_kv else 0
         self.o_width = self.n_heads * self.value_dim
-        self.w_in = self.w_o = self.slopes = None
+        self.w_in = self.w_o = self.slopes = self.sinks = None
         self.window_chunk = 1
+
+    @staticmethod
+    def shared_kv_given(p) -> bool:
+        return bool(p.get("shared_kv", False)) or bool(p.get("shares_packed", False))
 
     # ---- weights ----------------------------------------------------------
     def _n(self, which: str) -> str:
@@ -140,6 +160,10 @@ class SoftmaxAttention(Mixer):
             specs.append(WeightSpec(self._n("q_norm"), (H * d,), "norm_scale"))
             if not self.shared_kv:
                 specs.append(WeightSpec(self._n("k_norm"), (G * d,), "norm_scale"))
+        if self.qk_norm_weights:
+            specs += [WeightSpec(self._n("q_norm"), (d,), "norm_scale"), WeightSpec(self._n("k_norm"), (d,), "norm_scale")]
+        if self.sink == "learned":
+            specs.append(WeightSpec(self._n("sink"), (H,), "sink"))
         if self.output_gate:
             specs.append(WeightSpec(self._n("gate"), (H * e, self.hidden), "matrix"))
         specs.append(WeightSpec(self._n("out"), (self.hidden, H * e), "matrix"))
@@ -181,6 +205,16 @@ class SoftmaxAttention(Mixer):
             self.q_norm_w = padded("q_norm", self.n_heads)
             if not self.shared_kv:
                 self.k_norm_w = padded("k_norm", self.n_kv_heads)
+        elif self.qk_norm_weights:
+            def one_head(name):
+                out = torch.zeros(self.key_dim, dtype=torch.float32, device=self.w_in.device)
+                out[:self.key_dim_given] = float32_vector(tensors[self._n(name)])
+                return out
+            self.q_norm_w, self.k_norm_w = one_head("q_norm"), one_head("k_norm")
+        if self.sink == "learned":
+            self.sinks = float32_vector(tensors[self._n("sink")])
+        elif self.sink:
+            self.sinks = torch.zeros(self.n_heads, dtype=torch.float32, device=self.w_in.device)
         self.g_col = self.q_width + self.k_width + self.v_width
         if self.slope_exponent is not None:
             h = torch.arange(1, self.n_heads + 1, dtype=torch.float64)
@@ -214,21 +248,28 @@ class SoftmaxAttention(Mixer):
             return
         ring_tokens = ring_pages_for(self.cache_window, self.window_chunk - 1) * PAGE_TOKENS
         longest = max(step_lens)
-        if longest > ring_tokens - self.window + 1:
+        if longest > ring_tokens - self.span + 1:
             raise kernels.KernelError(
                 f"a layer with a window of {self.cache_window} keeps {ring_tokens} keys per sequence and cannot continue "
-                f"a sequence by {longest} tokens in one step (at most {ring_tokens - self.window + 1}; the engine's "
+                f"a sequence by {longest} tokens in one step (at most {ring_tokens - self.span + 1}; the engine's "
                 f"window_chunk option sets this)")
 
     # ---- one step -----------------------------------------------------------
+    def input_rows(self):
+        return self.w_in, None
+
     def forward(self, x, ctx: StepContext, residual):
-        b, kv, dev = ctx.batch, ctx.kv, x.device
-        T = x.shape[0]
+        proj = kernels.linear(x, self.w_in, out_dtype=torch.float32)
+        kernels.mark("qkv")
+        self.run(proj, ctx, residual, accumulate=not ctx.store_result)
+
+    def run(self, proj, ctx: StepContext, residual, accumulate: bool) -> None:
+        """The mixer on its projected rows (float32 [T, input rows], may be a column slice of wider rows)."""
+        b, kv, dev = ctx.batch, ctx.kv, proj.device
+        T = proj.shape[0]
         act = ctx.runtime.act_dtype
         owns = kv is not None and kv.writes and not self.shared_kv
         packed = self._use_packed(b.host_start, b.host_lens, owns)
-        proj = kernels.linear(x, self.w_in, out_dtype=torch.float32)
-        kernels.mark("qkv")
         q = torch.empty((T, self.q_width), dtype=act, device=dev)
         k = v = None
         if packed and self.shared_kv:
@@ -248,7 +289,7 @@ class SoftmaxAttention(Mixer):
             proj, (b.tok_pos, b.tok_seq, b.new_lens), q, q_col=0, k_col=self.k_col, v_col=self.v_col,
             n_heads=self.n_heads, n_kv_heads=0 if self.shared_kv else self.n_kv_heads, key_dim=self.key_dim,
             value_dim=self.value_dim, row_inv=row_inv, q_weight=self.q_norm_w, k_weight=self.k_norm_w,
-            paired=pos is not None and pos.paired,
+            paired=pos is not None and pos.paired, v_scale=self.result_scale,
             cos=pos.cos if pos is not None else None, sin=pos.sin if pos is not None else None,
             rotary_dim=pos.rotary_dim if pos is not None else 0, norm_eps=self.qk_norm_eps,
             k_out=None if self.shared_kv else k, v_out=None if self.shared_kv else v,
@@ -260,12 +301,13 @@ class SoftmaxAttention(Mixer):
         common = dict(n_heads=self.n_heads, n_kv_heads=self.n_kv_heads, key_dim=self.key_dim,
                       value_dim=self.value_dim, tok_pos=b.tok_pos, tok_seq=b.tok_seq, cu_seqlens=b.cu_seqlens,
                       start_pos=b.start_pos, scale=self.scale, window=self.window, keep_first=self.keep_first,
-                      softcap=self.softcap, slopes=self.slopes, sink=self.sink,
+                      softcap=self.softcap, slopes=self.slopes, chunk=self.chunk,
+                      sink=self.sinks if self.sinks is not None else False,
                       gate=proj[:, self.g_col:self.g_col + self.o_width] if self.output_gate else None)
         if packed:
             kernels.attention_ext(q, out, k_packed=k, v_packed=v, **common)
         else:
-            max_keys = b.max_new_len if self.window is None else min(b.max_new_len, self.window + self.keep_first)
+            max_keys = b.max_new_len if self.span is None else min(b.max_new_len, self.span + self.keep_first)
             n_splits = kernels.plan_splits(T, self.n_kv_heads, max_keys, ctx.runtime.sm_count)
             scratch = None
             if n_splits > 1:
@@ -275,5 +317,5 @@ class SoftmaxAttention(Mixer):
                                   table_width=kv.table_width, ring_pages=kv.ring_pages, page_tokens=kv.page_tokens,
                                   n_splits=n_splits, scratch=scratch, **common)
         kernels.mark("attention")
-        kernels.linear(out, self.w_o, out=residual, accumulate=not ctx.store_result)
+        kernels.linear(out, self.w_o, out=residual, accumulate=accumulate)
         kernels.mark("o")
