@@ -180,5 +180,5 @@ def write_safetensors(path: str, specs: list[tuple[str, torch.dtype, tuple[int, 
                     f"write_safetensors: expected '{name}' {dt} {shape}, got '{got_name}' {t.dtype} {tuple(t.shape)}")
             t = t.detach().contiguous().cpu()
             if t.numel():
-                f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() < (1 << 26)
-                        else memoryview(t.view(torch.uint8).numpy()))
+                f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() < (1 << 26)
+                        else memoryview(t.reshape(-1).view(torch.uint8).numpy()))
