@@ -26,12 +26,13 @@ then 256 decode steps.  Peaks come from MEASURED_PEAKS.json beside this file
 if it exists, else from an earlier measurement on the same kind of machine
 (6.65 TB/s, 1.59 PFLOP/s).
 
-`--design zodosun|rirudra|pavisun|furesun [--sizes 1k,2k,4k] [--prompt 2048]` is another program: the named decoder beside the Qwen2
+`--design zodosun|rirudra|pavisun|furesun|gokapel [--sizes 1k,2k,4k] [--prompt 2048]` is another program: the named decoder beside the Qwen2
 decoder of the same width, depth, heads, feed-forward and vocabulary (random weights, bfloat16): device time of a
 prompt, of decode steps at batch 8 and 64, and the time by class of kernel with what the attention and scan
 kernels reach of their rooflines, as one JSON line of its own (`--design rirudra` also runs the Zodosun decoder,
 whose scans are the like kernels of its own; `--design pavisun` runs the Pavisun decoder and the Qwen2 decoder only;
-`--design furesun` runs the Furesun, Rirudra and Qwen2 decoders).  The default workload and its line are untouched.
+`--design furesun` runs the Furesun, Rirudra and Qwen2 decoders; `--design gokapel` the Gokapel, Rirudra, Pavisun and
+Qwen2 decoders).  The default workload and its line are untouched.
 
 The reference arm (`--impl reference`) cannot run here: the reference is a
 Rust workspace and no Rust toolchain is installed, so it prints its
@@ -279,6 +280,103 @@ def furesun_config(width: int, ff: int, layers: int, vocab: int) -> dict:
             "max_positions": 8192, "layers": [order[i] for i in range(min(layers, 4))]}
 
 
+GOKAPEL_CHUNK, GOKAPEL_EXPERTS, GOKAPEL_TOP, GOKAPEL_STREAMS, GOKAPEL_RANK = 1024, 8, 2, 2, 128
+
+
+def gokapel_config(width: int, ff: int, layers: int, vocab: int) -> dict:
+    """A Gokapel configuration of the given width, heads of 128: the delta rule with a decay per key channel (half as
+    many key heads, two-step projections of inner width 128); attention in chunks of 1,024 on a quarter as many key
+    heads beside a minGRU as wide as the model; feed-forwards without a gate, half again as wide as the gated ones of
+    the other decoders (as many weights), dense in the first and last layer, in the second and third as 8 experts of a
+    quarter of that in 4 groups, of which a token uses 2 of 2 groups, and a shared one of half; 2 residual streams."""
+    heads, kv = width // 128, max(1, width // 512)
+    f = 3 * ff // 2
+    plain = {"kind": "dense", "ff": f}
+    moe = {"kind": "moe", "expert": {"ff": f // 4}, "shared": {"ff": f // 2},
+           "router": {"experts": GOKAPEL_EXPERTS, "top": GOKAPEL_TOP, "groups": {"count": 4, "keep": 2}}}
+    delta = {"heads": heads, "kv_heads": max(1, heads // 2), "dim": 128, "vdim": 128, "conv": 4,
+             "decay_rank": GOKAPEL_RANK, "gate_rank": GOKAPEL_RANK}
+    side = {"left": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                     "mask": {"size": GOKAPEL_CHUNK}, "rot": {"base": 1e6, "dims": 64}},
+            "left_scale": 0.7, "right": {"width": width}, "right_scale": 0.7}
+    order = [("channel_delta", delta, plain), ("parallel", side, moe), ("channel_delta", delta, moe), ("parallel", side, plain)]
+    return {"architecture": "Gokapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": GOKAPEL_STREAMS,
+            "residual_mult": 0.7, "embedding": {"scale": 8.0}, "max_positions": 8192,
+            "layers": [{"type": t, "mixer": m, "mlp": l} for t, m, l in (order[i % 4] for i in range(layers))]}
+
+
+def gokapel_roofline(rec: dict, pk: dict, P: int, sms: int) -> dict:
+    """What the classes of the Gokapel decoder reach of their rooflines, beside the like classes of the Rirudra decoder
+    (scan, convolution), of the Pavisun decoder (streams, experts) and of the Qwen2 decoder (attention, products)."""
+    width, ff, layers = rec["width"], rec["ff"], rec["layers"]
+    heads, kv, d = width // 128, max(1, width // 512), 128
+    g, r, p, q = rec["gokapel"], rec["rirudra"], rec["pavisun"], rec["qwen2"]
+    f, n_delta = 3 * ff // 2, 2
+    fp32_tflops = 2 * FP32_FMA_PER_SM_PER_CLOCK * sms * 1900.0 * 1e6 / 1e12
+    roof = {"fp32_fma_tflops_nominal": round(fp32_tflops, 1)}
+
+    def us(model, when, names):
+        return sum(model[when].get(k, 0.0) for k in names) * 1e-6
+
+    def tensor(name, flops, model, when, names):
+        roof[name + ".frac_of_bf16"] = round(flops / us(model, when, names) / 1e12 / pk["bf16_tflops"], 3)
+
+    def hbm(name, nbytes, model, when, names):
+        roof[name + ".frac_of_hbm"] = round(nbytes / us(model, when, names) / 1e9 / pk["hbm_gbs"], 3)
+
+    pre, dec = "prefill_classes_us", "decode_b64_classes_us"
+    C = GOKAPEL_CHUNK
+    tensor("gokapel.prefill.attention", 4 * heads * d * sum(i % C + 1 for i in range(P)) * 2, g, pre, ["attention"])
+    tensor("qwen2.prefill.attention", 4 * heads * d * P * (P + 1) / 2 * layers, q, pre, ["attention"])
+    seen = sum(min(i + 1, PAVISUN_WINDOW) for i in range(P))
+    tensor("pavisun.prefill.attention", 4 * heads * d * seen * layers, p, pre, ["attention"])
+    # delta rules: per token and head 8 d e operations; the state-space layer of the Rirudra decoder 5 d e
+    delta_state, ssm_state = heads * 128 * 128, (2 * width // 64) * 128 * 64
+    roof["gokapel.prefill.scan.frac_of_fp32_fma"] = round(P * 8 * delta_state * n_delta / us(g, pre, ["scan"]) / 1e12 / fp32_tflops, 3)
+    roof["rirudra.prefill.scan.frac_of_fp32_fma"] = round(
+        P * (5 * ssm_state + 8 * delta_state) / us(r, pre, ["scan"]) / 1e12 / fp32_tflops, 3)
+    hbm("gokapel.decode_b64.scan", 64 * delta_state * 4 * 2 * n_delta, g, dec, ["scan"])
+    hbm("rirudra.decode_b64.scan", 64 * (ssm_state + delta_state) * 4 * 2, r, dec, ["scan"])
+    # convolutions: float32 channels read and written once
+    ch_g, ch_r = 2 * max(1, heads // 2) * 128 + heads * 128, (2 * width + 256) + 2 * max(1, heads // 2) * 128 + heads * 128
+    hbm("gokapel.prefill.conv", P * 8 * ch_g * n_delta, g, pre, ["conv"])
+    hbm("rirudra.prefill.conv", P * 8 * ch_r, r, pre, ["conv"])
+    # the minGRU: three float32 columns read, a bfloat16 one written; the two-step projections: two float32 results
+    # written, one read and written once more
+    hbm("gokapel.prefill.gru", P * width * (3 * 4 + 2) * 2, g, pre, ["gru"])
+    hbm("gokapel.prefill.decay", P * heads * 128 * (4 + 4 + 8) * n_delta, g, pre, ["decay"])
+    # between the sublayers: streams read and written, the sublayer's float32 result (and here its gate) read, a rounded
+    # norm written
+    S = GOKAPEL_STREAMS
+    hbm("gokapel.prefill.between_sublayers", P * width * (8 * S + 4 + 4 + 2) * 2 * layers, g, pre, ["norms"])
+    S = PAVISUN_STREAMS
+    hbm("pavisun.prefill.between_sublayers", P * width * (8 * S + 4 + 2) * 2 * layers, p, pre, ["norms"])
+    # products: everything that reads a mixer's input, and the output products
+    n_in = [2 * max(1, heads // 2) * 128 + heads * 128 + width + 2 * GOKAPEL_RANK + heads, (heads + 2 * kv) * 128 + 4 * width]
+    tensor("gokapel.prefill.qkv", 2 * P * width * sum(n_in) * 2, g, pre, ["qkv"])
+    tensor("qwen2.prefill.qkv", 2 * P * width * (heads + 2 * kv) * 128 * layers, q, pre, ["qkv"])
+    tensor("gokapel.prefill.o", 2 * P * width * (heads * 128 * 4 + 2 * width), g, pre, ["o"])
+    tensor("qwen2.prefill.o", 2 * P * width * heads * 128 * layers, q, pre, ["o"])
+    tensor("gokapel.prefill.dense_feed_forward", 4 * P * width * f * 2, g, pre, ["up", "down"])
+    tensor("qwen2.prefill.dense_feed_forward", 6 * P * width * ff * layers, q, pre, ["gate_up", "down"])
+    tensor("gokapel.prefill.experts", 4 * P * width * (f // 4) * GOKAPEL_TOP * 2, g, pre, ["experts"])
+    tensor("pavisun.prefill.experts", 6 * P * width * (ff // PAVISUN_TOP) * PAVISUN_TOP * layers, p, pre, ["experts"])
+    tensor("gokapel.prefill.shared_expert", 4 * P * width * (f // 2) * 2, g, pre, ["shared_expert"])
+    tensor("gokapel.prefill.residual_gate_and_router", 2 * P * width * width * layers, g, pre, ["residual_gate", "router"])
+    hbm("gokapel.decode_b64.attention", 64 * ((P + 16) % C + 1) * 2 * kv * d * 2 * 2, g, dec, ["attention"])
+    hbm("qwen2.decode_b64.attention", 64 * (P + 16) * 2 * kv * d * 2 * layers, q, dec, ["attention"])
+    hbm("gokapel.decode_b64.products", 2 * width * (sum(n_in) * 2 + heads * 128 * 4 + 2 * width), g, dec, ["qkv", "o"])
+    hbm("qwen2.decode_b64.products", 2 * width * ((heads + 2 * kv) * 128 + heads * 128) * layers, q, dec, ["qkv", "o"])
+    hbm("gokapel.decode_b64.dense_feed_forward", 2 * width * f * 2 * 2, g, dec, ["up", "down"])
+    hbm("qwen2.decode_b64.dense_feed_forward", 3 * width * ff * 2 * layers, q, dec, ["gate_up", "down"])
+    hbm("gokapel.decode_b64.experts", 2 * width * (f // 4) * GOKAPEL_EXPERTS * 2 * 2, g, dec, ["experts"])
+    hbm("pavisun.decode_b64.experts", 3 * width * (ff // PAVISUN_TOP) * PAVISUN_EXPERTS * 2 * layers, p, dec, ["experts"])
+    hbm("gokapel.decode_b64.shared_expert", 2 * width * (f // 2) * 2 * 2, g, dec, ["shared_expert"])
+    hbm("gokapel.decode_b64.between_sublayers", 64 * width * (8 * GOKAPEL_STREAMS + 10) * 2 * layers, g, dec, ["norms"])
+    hbm("pavisun.decode_b64.between_sublayers", 64 * width * (8 * PAVISUN_STREAMS + 6) * 2 * layers, p, dec, ["norms"])
+    return roof
+
+
 def furesun_roofline(rec: dict, pk: dict, P: int, sms: int) -> dict:
     """What the classes of the Furesun decoder reach of their rooflines, beside the like classes of the Qwen2
     decoder (attention, feed-forward, the kernels between the sublayers) and of the Rirudra decoder (the scan)."""
@@ -447,6 +545,10 @@ def design_compare(args) -> int:
             if args.design == "furesun":
                 models = [("furesun", furesun_config(width, ff, layers, vocab)),
                           ("rirudra", rirudra_config(width, ff, layers, vocab)), ("qwen2", qwen)]
+            if args.design == "gokapel":
+                models = [("gokapel", gokapel_config(width, ff, layers, vocab)),
+                          ("rirudra", rirudra_config(width, ff, layers, vocab)),
+                          ("pavisun", pavisun_config(width, ff, layers, vocab)), ("qwen2", qwen)]
             for model, cfg in models:
                 eng = tq.Engine.from_random(cfg, seed=0, dtype="bfloat16", max_slots=64, max_context=ctx,
                                             max_tokens=64 * ctx)
@@ -520,6 +622,9 @@ def design_compare(args) -> int:
             if args.design == "furesun":
                 rec["roofline"] = furesun_roofline(rec, pk, P, sms)
                 continue
+            if args.design == "gokapel":
+                rec["roofline"] = gokapel_roofline(rec, pk, P, sms)
+                continue
             # what the classes reach of their rooflines
             heads, d = width // 128, 128
             z, q = rec["zodosun"], rec["qwen2"]
@@ -552,7 +657,7 @@ def design_compare(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["zodosun", "rirudra", "pavisun", "furesun"],
+    ap.add_argument("--design", default=None, choices=["zodosun", "rirudra", "pavisun", "furesun", "gokapel"],
                     help="instead of the default workload: this design beside the Qwen2 decoder of equal size")
     ap.add_argument("--sizes", default="1k,2k,4k", help="with --design: which of the sizes 1k, 2k, 4k (the model's width)")
     ap.add_argument("--gpus", type=int, default=1)

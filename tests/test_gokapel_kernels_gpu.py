@@ -33,7 +33,8 @@ def _cu(lens):
 # ---- the delta rule with a decay per key channel -----------------------------------------------------------------
 @pytest.mark.parametrize("H,G,d,e,lens", [(6, 2, 20, 12, (1, 37, 2, 70)), (2, 2, 64, 64, (130,)), (4, 1, 128, 128, (33, 1, 9)),
                                           (3, 3, 18, 30, (5, 5)), (1, 1, 200, 40, (40,)), (32, 16, 128, 128, (12, 3, 20)),
-                                          (24, 8, 64, 256, (9, 17, 4, 2)), (4, 2, 33, 7, (19, 20))])
+                                          (24, 8, 64, 256, (9, 17, 4, 2)), (4, 2, 33, 7, (19, 20)),
+                                          (2, 1, 256, 20, (3, 6)), (16, 8, 128, 128, (70,)), (5, 5, 30, 100, (4, 8, 1, 63))])
 def test_the_channel_delta_scan_against_the_recurrence(H, G, d, e, lens):
     """A ragged batch with shuffled slots and states that are not zero, then every sequence continued token by token
     with the one-token kernel; sizes that take every form of the scan."""
@@ -88,6 +89,35 @@ def test_the_channel_delta_scan_against_the_recurrence(H, G, d, e, lens):
     assert torch.equal(dev_state[:, H * d * e:].cpu(), state[:, H * d * e:])
 
 
+def test_decays_made_from_their_logits_and_channels_that_fade_at_once():
+    """The scan that makes the decays itself gives what it gives for ready ones; decays of exactly zero and one, and of
+    1e-30 in every token, leave everything finite."""
+    from tq_kv_b200 import kernels
+    g = torch.Generator().manual_seed(8)
+    H, d, e, lens = 3, 40, 24, (23, 2, 41)
+    T, n = sum(lens), len(lens)
+    buf = torch.randn(T, 2 * H * d + H * e, generator=g)
+    buf[:, :2 * H * d] = pg.unit(buf[:, :2 * H * d].reshape(T, 2 * H, d)).reshape(T, -1)
+    z, bias, a_log = torch.randn(T, H * d, generator=g) * 3.0, torch.randn(H * d, generator=g), torch.randn(H, generator=g)
+    bias[:4] = torch.tensor([200.0, -200.0, 69.0, 30.0])
+    a_log[0] = 0.0
+    w = torch.exp(-torch.exp(a_log).repeat_interleave(d) * torch.nn.functional.softplus(z + bias)).double().float()
+    scal = torch.sigmoid(torch.randn(T, H, 4, generator=g))
+    outs = []
+    for kw, x in (({}, w), (dict(dt_bias=bias.to(DEV), a_log=a_log.to(DEV)), z)):
+        state = torch.zeros(n, H * d * e, device=DEV)
+        b = buf.to(DEV)
+        out = torch.empty((T, H * e), device=DEV)
+        kernels.channel_delta_scan(b[:, :H * d], b[:, H * d:2 * H * d], b[:, 2 * H * d:], x.to(DEV), scal.to(DEV), state, _cu(lens),
+                                   _ints(list(range(n))), out, n_seqs=n, heads=H, qk_heads=H, key_dim=d, value_dim=e, **kw)
+        assert torch.isfinite(out).all() and torch.isfinite(state).all()
+        outs.append(out)
+    _close(outs[1], outs[0], 1e-5, "decays made inside")
+    want = pg.delta_scan(*(x.double() for x in (buf[:23, :H * d].reshape(23, H, d), buf[:23, H * d:2 * H * d].reshape(23, H, d),
+                                                buf[:23, 2 * H * d:].reshape(23, H, e), w[:23].reshape(23, H, d), scal[:23, :, 1])))
+    _close(outs[0][:23], want.reshape(23, -1), 2e-5, "first sequence")
+
+
 def test_write_strengths_beside_the_convolution():
     from tq_kv_b200 import kernels
     g = torch.Generator().manual_seed(3)
@@ -123,7 +153,8 @@ def test_the_two_step_projections(T, ra, rg, H, d, n, dtype):
     args = (ld[:, 3:3 + ra], wa.to(DEV), bias.to(DEV), a_log.to(DEV), ld[:, 3 + ra:3 + ra + rg], wg.to(DEV))
     tc = dtype == torch.bfloat16 and T >= 65 and min(ra, rg) >= 64
     for use_tc in (None, False):
-        decay, gate = kernels.low_rank_gates(*args, use_tc=use_tc)
+        decay, gate, done = kernels.low_rank_gates(*args, use_tc=use_tc)
+        assert done
         on_tc = tc and use_tc is None
         la, lg = (t.to(torch.bfloat16).double() if on_tc else t.double() for t in (low[:, 3:3 + ra], low[:, 3 + ra:3 + ra + rg]))
         z = la @ wa.double().T + bias.double()

@@ -12,7 +12,8 @@
 //                (the delta rule with one decay and one write strength per head and token: the state first
 //                fades, then what it holds along k_t is replaced by v_t at the rate beta_t)
 //   SCAN_CHANNEL_DELTA   S' = diag(w_t) S_{t-1};  u = beta_t (v_t - S'^T k_t);  S_t = S' + k_t u^T
-//                (as SCAN_GATED_DELTA with a decay per key channel; w ready-made, per head; keys as they are given)
+//                (as SCAN_GATED_DELTA with a decay per key channel; w ready-made, per head; one token per sequence only:
+//                many tokens are channel_scan.cu's)
 //   o_t = S_t^T q_t  in all.  The last three take their per-token scalars ready-made ([T, H, 4] floats: g, then
 //   dt or beta; SCAN_CHANNEL_DELTA reads beta only), the value columns may be narrower or wider than the keys, and head h reads the q/k vectors of
 //   head h / qk_div.
@@ -43,7 +44,6 @@
 #define SCAN_GATED 2
 #define SCAN_GATED_DELTA 3
 #define SCAN_CHANNEL_DELTA 4
-#define SCAN_VECTORS(MODE) ((MODE) == SCAN_DELTA ? 5 : ((MODE) == SCAN_CHANNEL_DELTA ? 3 : 2))      // per token, of d each
 #define SCAN_THREADS 128      // of the one-token kernel
 
 struct ScanArgs {
@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(THREADS) linear_scan_kernel(ScanArgs a) {
     constexpr int RK = 8;
     constexpr int DP = KG * RK;
     constexpr int CT = THREADS / KG * RC;
-    constexpr int NV = SCAN_VECTORS(MODE);
+    constexpr int NV = MODE == SCAN_DELTA ? 5 : 2;
     constexpr int SC = MODE >= SCAN_GATED ? 4 : 0;          // a token's scalars, in front of a stage
     // tokens whose instructions the compiler may interleave (measured: the rules with one decay per head gain
     // up to 10 % from four, 2,048 tokens of 16 heads of 128 x 128: 716 -> 643 us)
@@ -166,7 +166,7 @@ __global__ void __launch_bounds__(THREADS) linear_scan_kernel(ScanArgs a) {
     const float skip = (MODE == SCAN_GATED && a.skip) ? a.skip[head] : 0.f;
     __syncthreads();
 
-    // stage s holds, token by token: q[DP] k[DP] (u[DP] au[DP] w[DP], or w[DP]) and after all of them v[TC][CT]
+    // stage s holds, token by token: q[DP] k[DP] (u[DP] au[DP] w[DP]) and after all of them v[TC][CT]
     auto stage_in = [&](int base, int s) {
         const int n = min(TC, t1 - base);
         float* dsc = sm + s * stage_floats;
@@ -195,7 +195,6 @@ __global__ void __launch_bounds__(THREADS) linear_scan_kernel(ScanArgs a) {
                     cp_async16(row + 3 * DP, a.au + t * a.ldp + head * d + i);
                     cp_async16(row + 4 * DP, a.w + t * a.ldw + head * d + i);
                 }
-                if (MODE == SCAN_CHANNEL_DELTA) cp_async16(row + 2 * DP, a.w + t * a.ldw + head * d + i);
             }
             if (CT % 4 == 0) {                 // (a block of fewer than four columns takes its values one by one, below)
                 for (int idx = tid; idx < n * c4; idx += THREADS) {
@@ -215,7 +214,6 @@ __global__ void __launch_bounds__(THREADS) linear_scan_kernel(ScanArgs a) {
                     row[3 * DP] = a.au[t * a.ldp + head * d + i];
                     row[4 * DP] = a.w[t * a.ldw + head * d + i];
                 }
-                if (MODE == SCAN_CHANNEL_DELTA) row[2 * DP] = a.w[t * a.ldw + head * d + i];
             }
         }
         if (!a.vec || CT % 4 != 0) {
@@ -322,39 +320,6 @@ __global__ void __launch_bounds__(THREADS) linear_scan_kernel(ScanArgs a) {
                         o2[c] = __ffma2_rn(qq[r], S[r][c], o2[c]);
                     }
                 }
-            } else if (MODE == SCAN_CHANNEL_DELTA) {
-                const float beta = ssc[tt * 4 + 1];
-                float2 ww[RK / 2], wk[RK / 2];
-#pragma unroll
-                for (int g = 0; g < 2; ++g) {
-                    const float4 w4 = pq[2 * (DP / 4) + g * KG];
-                    ww[2 * g] = make_float2(w4.x, w4.y); ww[2 * g + 1] = make_float2(w4.z, w4.w);
-                }
-#pragma unroll
-                for (int r = 0; r < RK / 2; ++r) wk[r] = __fmul2_rn(ww[r], kk[r]);      // (diag(w) S)^T k = S^T (w * k)
-                float dot[RC];
-#pragma unroll
-                for (int c = 0; c < RC; ++c) {
-                    float2 acc = __fmul2_rn(wk[0], S[0][c]);
-#pragma unroll
-                    for (int r = 1; r < RK / 2; ++r) acc = __ffma2_rn(wk[r], S[r][c], acc);
-                    dot[c] = acc.x + acc.y;
-                }
-#pragma unroll
-                for (int off = KG / 2; off > 0; off >>= 1) {
-#pragma unroll
-                    for (int c = 0; c < RC; ++c) dot[c] += __shfl_xor_sync(0xffffffffu, dot[c], off);
-                }
-#pragma unroll
-                for (int c = 0; c < RC; ++c) {
-                    const float u = beta * (xr[c] - dot[c]);
-                    const float2 uu = make_float2(u, u);
-#pragma unroll
-                    for (int r = 0; r < RK / 2; ++r) {
-                        S[r][c] = __ffma2_rn(ww[r], S[r][c], __fmul2_rn(kk[r], uu));
-                        o2[c] = __ffma2_rn(qq[r], S[r][c], o2[c]);
-                    }
-                }
             } else {
                 float2 cc = make_float2(c_head, c_head);
                 if (MODE == SCAN_GATED) {
@@ -424,7 +389,7 @@ __global__ void __launch_bounds__(THREADS) linear_scan_kernel(ScanArgs a) {
 
 template <int MODE, int KG, int THREADS, int RC>
 static int launch_scan(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
-    constexpr int CT = THREADS / KG * RC, DP = KG * 8, NV = SCAN_VECTORS(MODE), SC = MODE >= SCAN_GATED ? 4 : 0;
+    constexpr int CT = THREADS / KG * RC, DP = KG * 8, NV = MODE == SCAN_DELTA ? 5 : 2, SC = MODE >= SCAN_GATED ? 4 : 0;
     ScanArgs args = a;
     const int per_token = 2 * (SC + NV * DP + CT) + CT;  // two stages and the outputs
     int chunk = 8;
@@ -663,20 +628,18 @@ TQ_API int tq_gated_scan(int delta, const float* q, const float* k, const float*
     return dispatch_scan<SCAN_GATED>(a, n_seqs, stream);
 }
 
-// The delta rule with a decay per head and key channel: as tq_gated_scan with `delta`, but the decays are w [T, ldw]
-// (head h's d channels from column h * d) and of scal only the write strength (entry 1) is read.
-TQ_API int tq_channel_delta_scan(const float* q, const float* k, const float* v, int ldp, const float* w, int ldw,
+// One token of every sequence through the delta rule with a decay per head and key channel: as tq_gated_scan with
+// `delta` and `single`, but the decays are w [n_seqs, ldw] (head h's d channels from column h * d) and of scal only the
+// write strength (entry 1) is read.
+TQ_API int tq_channel_delta_step(const float* q, const float* k, const float* v, int ldp, const float* w, int ldw,
                                  const float* scal, int qk_div, float* state, long long state_stride,
-                                 const int* cu_seqlens, const int* slots, int n_seqs, int n_tokens, int single, float* out,
-                                 int ldo, int H, int d, int e, cudaStream_t stream) {
-    if (n_seqs <= 0 || n_tokens <= 0) return 0;
+                                 const int* cu_seqlens, const int* slots, int n_seqs, float* out, int ldo, int H, int d,
+                                 int e, cudaStream_t stream) {
+    if (n_seqs <= 0) return 0;
     if (!q || !k || !v || !w || !scal || !state || !cu_seqlens || !slots || !out || H <= 0 || H > 65535 || d <= 0 || d > 256 ||
         e <= 0 || qk_div <= 0 || H % qk_div || state_stride < (long long)H * d * e || ldw < H * d)
         return (int)cudaErrorInvalidValue;
     ScanArgs a{q, k, v, nullptr, ldp, nullptr, 0, w, ldw, nullptr, state, cu_seqlens, slots, out, ldo, H, d, e, 0, 0,
                0, 0.f, scal, nullptr, qk_div, (size_t)state_stride};
-    auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    a.vec = (d % 4 == 0 && e % 4 == 0 && ldp % 4 == 0 && ldw % 4 == 0 && al(q) && al(k) && al(v) && al(w) && al(scal)) ? 1 : 0;
-    if (single) return dispatch_step<SCAN_CHANNEL_DELTA>(a, n_seqs, stream);
-    return dispatch_scan<SCAN_CHANNEL_DELTA>(a, n_seqs, stream);
+    return dispatch_step<SCAN_CHANNEL_DELTA>(a, n_seqs, stream);
 }

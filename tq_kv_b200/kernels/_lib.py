@@ -183,9 +183,11 @@ _SIGNATURES = {
     "tq_add_scaled": [c_void_p, c_void_p, c_size_t, c_float, c_void_p],
     "tq_gated_scan": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, ctypes.c_longlong,
                       c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-    "tq_channel_delta_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
-                              ctypes.c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
-                              c_int, c_void_p],
+    "tq_channel_delta_step": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
+                              ctypes.c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "tq_channel_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                        c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                        c_void_p],
     "tq_short_conv": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, ctypes.c_longlong, c_void_p,
                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                       c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
@@ -278,5 +280,7 @@ def core() -> ctypes.CDLL:
             fn = getattr(lib, name)
             fn.argtypes = argtypes
             fn.restype = c_int
+        lib.tq_channel_scan_floats.argtypes = [c_int, c_int, c_int, c_int]
+        lib.tq_channel_scan_floats.restype = ctypes.c_longlong
         _core = lib
     return _core

@@ -24,10 +24,12 @@ def round_columns(x: torch.Tensor) -> torch.Tensor:
 
 
 def low_rank_gates(low_decay: torch.Tensor, w_decay: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
-                   low_gate: torch.Tensor, w_gate: torch.Tensor, *, use_tc: Optional[bool] = None):
+                   low_gate: torch.Tensor, w_gate: torch.Tensor, *, use_tc: Optional[bool] = None, leave_logits: bool = False):
     """The second halves of two two-step projections whose first halves are columns of one float32 buffer:
     decay[t, i] = exp(-exp(a_log[i // d]) * softplus(w_decay[i] . low_decay[t] + dt_bias[i])), d = len(dt_bias) //
-    len(a_log), and gate[t, i] = w_gate[i] . low_gate[t]; both float32 [T, n].  The weights share one dtype."""
+    len(a_log), and gate[t, i] = w_gate[i] . low_gate[t]; both float32 [T, n].  The weights share one dtype.  Returns
+    (decay, gate, done): with `leave_logits` the decays may be left as w_decay . low_decay, for a reader that makes them
+    itself; `done` then is False."""
     T = low_decay.shape[0]
     na, ra = w_decay.shape
     np_, rp = w_gate.shape
@@ -45,11 +47,13 @@ def low_rank_gates(low_decay: torch.Tensor, w_decay: torch.Tensor, dt_bias: torc
                   and ra % 8 == 0 and rp % 8 == 0)
     if use_tc:
         decay = linear(round_columns(low_decay), w_decay, out_dtype=torch.float32)
-        check(core().tq_channel_decay(ptr(decay), ptr(dt_bias), ptr(a_log), d, na, T, stream()), "channel_decay")
-        return decay, linear(round_columns(low_gate), w_gate, out_dtype=torch.float32)
+        gate = linear(round_columns(low_gate), w_gate, out_dtype=torch.float32)
+        if not leave_logits:
+            check(core().tq_channel_decay(ptr(decay), ptr(dt_bias), ptr(a_log), d, na, T, stream()), "channel_decay")
+        return decay, gate, not leave_logits
     decay = torch.empty((T, na), dtype=torch.float32, device=low_decay.device)
     gate = torch.empty((T, np_), dtype=torch.float32, device=low_decay.device)
     check(core().tq_low_rank_rows(ptr(low_decay), ra, ptr(w_decay), na, ptr(dt_bias), ptr(a_log), d, ptr(decay),
                                   ptr(low_gate), rp, ptr(w_gate), np_, ptr(gate), low_decay.stride(0), dtype_code(w_decay),
                                   T, stream()), "low_rank_rows")
-    return decay, gate
+    return decay, gate, True

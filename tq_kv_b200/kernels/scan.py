@@ -184,10 +184,12 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scalars: torch
 
 def channel_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor,
                        state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, out: torch.Tensor, *,
-                       n_seqs: int, heads: int, qk_heads: int, key_dim: int, value_dim: int, single_tokens: bool = False):
+                       n_seqs: int, heads: int, qk_heads: int, key_dim: int, value_dim: int, single_tokens: bool = False,
+                       dt_bias: Optional[torch.Tensor] = None, a_log: Optional[torch.Tensor] = None):
     """The delta rule with a decay per head and key channel:  S' = diag(w) S;  S = S' + k (beta (v - S'^T k))^T;
-    o = S^T q.  Operands as in `gated_scan`; `decay` float32 [T, heads * d] holds w, of `scalars` only beta (entry 1)
-    is read."""
+    o = S^T q (csrc/channel_scan.cu; one token per sequence: csrc/linear_scan.cu).  Operands as in `gated_scan`; `decay`
+    float32 [T, heads * d] holds w — or, with dt_bias [heads * d] and a_log [heads] (not with `single_tokens`), z of
+    w = exp(-exp(a_log) softplus(z + dt_bias)) — and of `scalars` only beta (entry 1) is read."""
     T = q.shape[0]
     d, e = int(key_dim), int(value_dim)
     for name, t, n in (("q", q, qk_heads * d), ("k", k, qk_heads * d), ("v", v, heads * e)):
@@ -204,11 +206,22 @@ def channel_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay:
         raise KernelError("channel_delta_scan: state must be float32 [slots, >= heads * d * e]")
     if out.dtype != torch.float32 or tuple(out.shape) != (T, heads * e) or out.stride(1) != 1:
         raise KernelError("channel_delta_scan: out must be float32 [T, heads * e]")
-    if single_tokens and T != n_seqs:
-        raise KernelError("channel_delta_scan: single_tokens needs one token per sequence")
-    need_contiguous(cu_seqlens=cu_seqlens, slots=slots)
-    check(core().tq_channel_delta_scan(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(decay), decay.stride(0), ptr(scalars),
-                                       heads // qk_heads, ptr(state), state.stride(0), ptr(cu_seqlens), ptr(slots),
-                                       int(n_seqs), T, int(single_tokens), ptr(out), out.stride(0), heads, d, e, stream()),
-          "channel_delta_scan")
+    if (dt_bias is None) != (a_log is None):
+        raise KernelError("channel_delta_scan: dt_bias and a_log come together")
+    if dt_bias is not None and (single_tokens or dt_bias.dtype != torch.float32 or tuple(dt_bias.shape) != (heads * d,)
+                                or a_log.dtype != torch.float32 or tuple(a_log.shape) != (heads,)):
+        raise KernelError("channel_delta_scan: dt_bias float32 [heads * d] and a_log float32 [heads], for many tokens")
+    need_contiguous(cu_seqlens=cu_seqlens, slots=slots, dt_bias=dt_bias, a_log=a_log)
+    lib = core()
+    if single_tokens:
+        if T != n_seqs:
+            raise KernelError("channel_delta_scan: single_tokens needs one token per sequence")
+        check(lib.tq_channel_delta_step(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(decay), decay.stride(0), ptr(scalars),
+                                        heads // qk_heads, ptr(state), state.stride(0), ptr(cu_seqlens), ptr(slots),
+                                        int(n_seqs), ptr(out), out.stride(0), heads, d, e, stream()), "channel_delta_step")
+        return out
+    rec = torch.empty(lib.tq_channel_scan_floats(T, int(n_seqs), heads, d), dtype=torch.float32, device=q.device)
+    check(lib.tq_channel_scan(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(decay), decay.stride(0), ptr(dt_bias), ptr(a_log),
+                              ptr(scalars), heads // qk_heads, ptr(rec), ptr(state), state.stride(0), ptr(cu_seqlens),
+                              ptr(slots), int(n_seqs), T, ptr(out), out.stride(0), heads, d, e, stream()), "channel_scan", 2)
     return out

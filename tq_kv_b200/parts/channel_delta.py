@@ -10,7 +10,7 @@
 conv is a short causal convolution over time per channel (no bias); unit(x) = x / sqrt(sum(x^2) + unit_eps) per head;
 head h reads the q and k of key head h // (heads / key_heads).  S starts at zero, is float32 and lives, with the
 convolutions' last taps - 1 inputs, in the cache's per-sequence state (csrc/short_conv.cu, csrc/low_rank.cu,
-csrc/linear_scan.cu).  Everything that reads h is one product with a float32 result, which may carry a rider's rows.
+csrc/channel_scan.cu; one token at a time csrc/linear_scan.cu).  Everything that reads h is one product with a float32 result, which may carry a rider's rows.
 """
 from __future__ import annotations
 
@@ -117,17 +117,19 @@ class ChannelDeltaMixer(Mixer):
                            silu=True, single_tokens=single, unit_eps=self.unit_eps,
                            beta_raw=proj[:, self.off_b:self.off_b + H], scalars=scal)
         kernels.mark("conv")
-        decay, gate = kernels.low_rank_gates(proj[:, self.off_a:self.off_g], self.w_decay, self.dt_bias, self.a_log,
-                                             proj[:, self.off_g:self.off_b], self.w_gate)
+        decay, gate, done = kernels.low_rank_gates(proj[:, self.off_a:self.off_g], self.w_decay, self.dt_bias, self.a_log,
+                                                   proj[:, self.off_g:self.off_b], self.w_gate,
+                                                   leave_logits=not single)
         kernels.mark("decay")
         o = torch.empty((T, vw), dtype=torch.float32, device=dev)
         kernels.channel_delta_scan(cv[:, :qk], cv[:, qk:2 * qk], cv[:, 2 * qk:], decay, scal,
                                    ctx.state[:, :self.state_floats], b.cu_seqlens, b.slots, o, n_seqs=b.n_seqs, heads=H,
                                    qk_heads=self.key_heads, key_dim=self.key_dim, value_dim=self.value_dim,
-                                   single_tokens=single)
+                                   single_tokens=single, dt_bias=None if done else self.dt_bias,
+                                   a_log=None if done else self.a_log)
         kernels.mark("scan")
         y = torch.empty((T, vw), dtype=ctx.runtime.act_dtype, device=dev)
         kernels.group_rmsnorm(o, self.norm_w, self.eps, y, groups=H, gate=gate)
-        kernels.mark("norms")
+        kernels.mark("head_norm")
         kernels.linear(y, self.w_o, out=residual, accumulate=not ctx.store_result)
         kernels.mark("o")

@@ -65,6 +65,6 @@ class MinGRUMixer(Mixer):
         y = torch.empty((proj.shape[0], n), dtype=ctx.runtime.act_dtype, device=proj.device)
         kernels.gru_scan(proj[:, :n], proj[:, s:s + n], proj[:, 2 * s:2 * s + n], ctx.state, b.cu_seqlens, b.slots, y,
                          n_seqs=b.n_seqs, scale=self.result_scale, single_tokens=b.single_tokens)
-        kernels.mark("scan")
+        kernels.mark("gru")
         kernels.linear(y, self.w_o, out=residual, accumulate=accumulate)
         kernels.mark("o")
