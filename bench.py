@@ -280,12 +280,12 @@ def furesun_config(width: int, ff: int, layers: int, vocab: int) -> dict:
             "max_positions": 8192, "layers": [order[i] for i in range(min(layers, 4))]}
 
 
-GOKAPEL_CHUNK, GOKAPEL_EXPERTS, GOKAPEL_TOP, GOKAPEL_STREAMS, GOKAPEL_RANK = 1024, 8, 2, 2, 128
+GOKAPEL_CHUNK, GOKAPEL_EXPERTS, GOKAPEL_TOP, GOKAPEL_STREAMS, GOKAPEL_RANK = 1100, 8, 2, 2, 128
 
 
 def gokapel_config(width: int, ff: int, layers: int, vocab: int) -> dict:
     """A Gokapel configuration of the given width, heads of 128: the delta rule with a decay per key channel (half as
-    many key heads, two-step projections of inner width 128); attention in chunks of 1,024 on a quarter as many key
+    many key heads, two-step projections of inner width 128); attention in chunks of 1,100 (a decoded token after 2,048 then sees about a thousand keys) on a quarter as many key
     heads beside a minGRU as wide as the model; feed-forwards without a gate, half again as wide as the gated ones of
     the other decoders (as many weights), dense in the first and last layer, in the second and third as 8 experts of a
     quarter of that in 4 groups, of which a token uses 2 of 2 groups, and a shared one of half; 2 residual streams."""

@@ -19,16 +19,15 @@
 //                   Fours start at each sequence's first token of the step; the last one of a sequence is filled up
 //                   with tokens that change nothing (w = 1, k = q = 0, beta = 0).
 // channel_scan      a block owns some columns of one head of one sequence and walks the records in order, every thread
-//                   4 (or 8) keys x 2 columns of the state in registers, the records through shared memory two stages
-//                   deep.
-//                   The eight products of two columns are summed over the lanes that share the columns by trading
+//                   4 (or 8) keys x 2 (or 4) columns of the state in registers, the records through shared memory two
+//                   stages deep.
+//                   The products of a thread's columns are summed over the lanes that share the columns by trading
 //                   halves of the values: each lane ends with the sums it needs to hand on.  grid (sequence, head,
 //                   column tile).
 #include "common.cuh"
 
 #define CS_TOKENS 4
 #define CS_SCALARS 40                     // a [4][4], b [4][4], beta [4], padding
-#define CS_RC 2                           // columns of a thread
 
 __host__ __device__ constexpr int cs_record(int dp) { return 13 * dp + CS_SCALARS; }
 // the first record of sequence b, whose first token is t0: leaves room for every sequence's part-filled last four
@@ -54,18 +53,18 @@ __device__ __forceinline__ void cs_cp16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(p), "l"(src) : "memory");
 }
 
-// Sums 16 values over N lanes (N = 4 .. 32, a power of two; `l`: the lane's place among them) by trading halves:
-// afterwards a lane holds the full sums of values l * (16 / N) .. (N >= 16: of value l / (N / 16)) in v[0 ..].
-template <int N>
-__device__ __forceinline__ void cs_trade_sums(float (&v)[16], int l) {
-    int count = 16;
+// Sums V values over N lanes (powers of two; `l`: the lane's place among them) by trading halves: afterwards a lane
+// holds the full sums of values l * (V / N) .. in v[0 ..] (N > V: of value l / (N / V)).
+template <int N, int V>
+__device__ __forceinline__ void cs_trade_sums(float (&v)[V], int l) {
+    int count = V;
 #pragma unroll
     for (int off = N / 2; off > 0; off >>= 1) {
         if (count > 1) {
             count >>= 1;
             const bool high = l & off;
 #pragma unroll
-            for (int i = 0; i < 8; ++i)
+            for (int i = 0; i < V / 2; ++i)
                 if (i < count) {
                     const float give = high ? v[i] : v[i + count], keep = high ? v[i + count] : v[i];
                     v[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
@@ -141,7 +140,7 @@ __global__ void __launch_bounds__(128) channel_prepare_kernel(ChannelArgs a) {
         for (int j = 0; j < CS_TOKENS; ++j) rec[(2 * CS_TOKENS + j) * a.dp + i0] = kt[j];
         rec[3 * CS_TOKENS * a.dp + i0] = run;
     }
-    cs_trade_sums<32>(sums, lane);                       // lanes 2 s and 2 s + 1 hold sum s
+    cs_trade_sums<32, 16>(sums, lane);                       // lanes 2 s and 2 s + 1 hold sum s
     float* sc = rec + 13 * a.dp;
     if (lane < 20) {                                     // what the sums leave out: zeros above the diagonals, beta
         const int i = lane & 15, row = i >> 2, col = i & 3;
@@ -165,12 +164,14 @@ __global__ void __launch_bounds__(128) channel_prepare_kernel(ChannelArgs a) {
     }
 }
 
-// KG lanes share two columns; each holds RK of their KG * RK (padded) keys.
-template <int KG, int RK, int THREADS>
+// KG lanes share RC columns; each holds RK of their KG * RK (padded) keys.
+template <int KG, int RK, int RC, int THREADS>
 __global__ void __launch_bounds__(THREADS) channel_scan_kernel(ChannelArgs a) {
-    constexpr int RC = CS_RC, DP = KG * RK, REC = cs_record(DP), R4 = RK / 4, R2 = RK / 2;
+    constexpr int DP = KG * RK, REC = cs_record(DP), R4 = RK / 4, R2 = RK / 2;
     constexpr int CT = THREADS / KG * RC;
-    constexpr int PER = KG >= 16 ? 1 : 16 / KG;          // sums a lane holds after trading
+    constexpr int V = 2 * CS_TOKENS * RC;                // sums per four tokens and thread
+    constexpr int PER = KG >= V ? 1 : V / KG;            // of which a lane holds this many after trading
+    constexpr int SAME = KG >= V ? KG / V : 1;           // and this many lanes hold the same
     extern __shared__ __align__(16) float sm[];
     const int b = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * CT;
     const int tid = threadIdx.x, kg = tid % KG, cg = tid / KG;
@@ -221,7 +222,7 @@ __global__ void __launch_bounds__(THREADS) channel_scan_kernel(ChannelArgs a) {
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
     // (where two lanes end with the same sum one of them hands it on)
-    const bool o_lane = KG <= 16 || kg % (KG / 16) == 0;
+    const bool o_lane = kg % SAME == 0;
 
     if (n4 > 0) stage_in(0, 0);
     int s = 0;
@@ -241,8 +242,8 @@ __global__ void __launch_bounds__(THREADS) channel_scan_kernel(ChannelArgs a) {
         for (int f = 0; f < n; ++f) {
             const float4* vecs = reinterpret_cast<const float4*>(src + f * REC) + kg;
             const float* sc = src + f * REC + 13 * DP;
-            // the products with the state: value (type << 3) | (token << 1) | column, type 0 keys, 1 queries
-            float r[16];
+            // the products with the state: value (type * 4 + token) * RC + column, type 0 keys, 1 queries
+            float r[V];
 #pragma unroll
             for (int type = 0; type < 2; ++type)
 #pragma unroll
@@ -259,22 +260,28 @@ __global__ void __launch_bounds__(THREADS) channel_scan_kernel(ChannelArgs a) {
                         }
                     }
 #pragma unroll
-                    for (int c = 0; c < RC; ++c) r[type * 8 + i * 2 + c] = acc[c].x + acc[c].y;
+                    for (int c = 0; c < RC; ++c) r[(type * CS_TOKENS + i) * RC + c] = acc[c].x + acc[c].y;
                 }
-            cs_trade_sums<KG>(r, kg);
-            // every lane takes the keys' products back and solves for the four u of both columns
+            cs_trade_sums<KG, V>(r, kg);
+            // every lane takes the keys' products back and solves for the four u of its columns
             const float4 a1 = *reinterpret_cast<const float4*>(sc + 4), a2 = *reinterpret_cast<const float4*>(sc + 8);
             const float4 a3 = *reinterpret_cast<const float4*>(sc + 12), be = *reinterpret_cast<const float4*>(sc + 32);
             float u[CS_TOKENS][RC], x[CS_TOKENS][RC];
 #pragma unroll
             for (int i = 0; i < CS_TOKENS; ++i) {
-                const float2 v = *reinterpret_cast<const float2*>(sv + (f * CS_TOKENS + i) * CT);
+                float v[RC];
+#pragma unroll
+                for (int c = 0; c < RC; c += 2) {
+                    const float2 two = *reinterpret_cast<const float2*>(sv + (f * CS_TOKENS + i) * CT + c);
+                    v[c] = two.x;
+                    v[c + 1] = two.y;
+                }
 #pragma unroll
                 for (int c = 0; c < RC; ++c) {
-                    const int id = i * 2 + c;
-                    const int src_lane = (tid & 31 & ~(KG - 1)) + (KG <= 16 ? id / PER : id * (KG / 16));
-                    const float dot = __shfl_sync(0xffffffffu, r[KG <= 16 ? id % PER : 0], src_lane);
-                    x[i][c] = (f * CS_TOKENS + i < left ? (c ? v.y : v.x) : 0.f) - dot;
+                    const int id = i * RC + c;
+                    const int src_lane = (tid & 31 & ~(KG - 1)) + id / PER * SAME;
+                    const float dot = __shfl_sync(0xffffffffu, r[id % PER], src_lane);
+                    x[i][c] = (f * CS_TOKENS + i < left ? v[c] : 0.f) - dot;
                 }
             }
 #pragma unroll
@@ -309,14 +316,22 @@ __global__ void __launch_bounds__(THREADS) channel_scan_kernel(ChannelArgs a) {
             // the lanes that hold the queries' products finish the results
 #pragma unroll
             for (int p = 0; p < PER; ++p) {
-                const int id = KG <= 16 ? kg * PER + p : kg / (KG / 16);
-                const int i = (id >> 1) & 3, c = id & 1, tok = f * CS_TOKENS + i;
+                const int id = kg / SAME * PER + p;
+                const int i = (id / RC) & 3, c = id % RC, tok = f * CS_TOKENS + i;
                 const float4 bi = *reinterpret_cast<const float4*>(sc + 16 + 4 * i);
-                float o = fmaf(bi.x, c ? u[0][1] : u[0][0], r[p]);
-                o = fmaf(bi.y, c ? u[1][1] : u[1][0], o);
-                o = fmaf(bi.z, c ? u[2][1] : u[2][0], o);
-                o = fmaf(bi.w, c ? u[3][1] : u[3][0], o);
-                if (id >= 8 && o_lane && tok < left && colb + c < e)
+                float uc[CS_TOKENS];                     // the u of column c (whose low part p fixes)
+#pragma unroll
+                for (int j = 0; j < CS_TOKENS; ++j) {
+                    uc[j] = u[j][p % RC];
+#pragma unroll
+                    for (int m = PER; m < RC; m += PER)
+                        if (c == m + p) uc[j] = u[j][(m + p) % RC];
+                }
+                float o = fmaf(bi.x, uc[0], r[p]);
+                o = fmaf(bi.y, uc[1], o);
+                o = fmaf(bi.z, uc[2], o);
+                o = fmaf(bi.w, uc[3], o);
+                if (id >= CS_TOKENS * RC && o_lane && tok < left && colb + c < e)
                     a.out[(size_t)(base + tok) * a.ldo + head * e + colb + c] = o;
             }
         }
@@ -331,38 +346,51 @@ __global__ void __launch_bounds__(THREADS) channel_scan_kernel(ChannelArgs a) {
     }
 }
 
-#define CS_SMEM_ALONE (116 * 1024)        // two such blocks do not fit the 228 KB of an SM (linear_scan.cu says why)
+#define CS_SMEM_ALONE (116 * 1024)        // the most a block asks for
+#define CS_SMEM_SM (230 * 1024)           // a little more than an SM has for all its blocks
 
-template <int KG, int RK, int THREADS>
+template <int KG, int RK, int RC, int THREADS>
 static int launch_channel_scan(const ChannelArgs& a, cudaStream_t stream) {
-    constexpr int CT = THREADS / KG * CS_RC, REC = cs_record(KG * RK);
+    constexpr int CT = THREADS / KG * RC, REC = cs_record(KG * RK);
     const dim3 grid(a.n_seqs, a.H, (a.e + CT - 1) / CT);
-    const bool alone = (long long)grid.x * grid.y * grid.z <= tq_sm_count();
+    // Blocks that start while the kernel before drains gather on the SMs that fall free first; so a block of a small
+    // grid asks for as much shared memory as lets no SM take more than its share of them.
+    const long long per_sm = ((long long)grid.x * grid.y * grid.z + tq_sm_count() - 1) / tq_sm_count();
     ChannelArgs args = a;
-    args.fours = alone && REC < 2000 ? 4 : 2;
+    args.fours = per_sm <= 2 && REC < 2000 ? 4 : 2;
     size_t smem = (size_t)2 * args.fours * (REC + CS_TOKENS * CT) * sizeof(float);
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(channel_scan_kernel<KG, RK, THREADS>,
+        cudaError_t e = cudaFuncSetAttribute(channel_scan_kernel<KG, RK, RC, THREADS>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, CS_SMEM_ALONE);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     if (smem > CS_SMEM_ALONE) return (int)cudaErrorInvalidValue;
-    if (alone) smem = CS_SMEM_ALONE;
-    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, channel_scan_kernel<KG, RK, THREADS>, grid, dim3(THREADS), smem, stream, args);
+    if (per_sm <= 4) {
+        const size_t share = (size_t)CS_SMEM_SM / (per_sm + 1);
+        if (smem < share) smem = share;
+    }
+    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, channel_scan_kernel<KG, RK, RC, THREADS>, grid, dim3(THREADS), smem, stream, args);
 }
 
+// Few sequences and heads: short chains count (four keys a thread, two columns), in blocks of eight warps while they
+// still give most SMs one, in smaller ones where columns are few.  Many: reads of shared memory count (eight keys, four
+// columns: a vector read serves twice the columns, its sums half the lanes).
 template <int KG, int RK>
 static int pick_channel_scan(const ChannelArgs& a, cudaStream_t stream) {
-    // blocks of eight warps while they still give most SMs one, smaller ones where columns are few
-    auto blocks = [&](int threads) {
-        const int ct = threads / KG * CS_RC;
+    auto blocks = [&](int kg, int rc, int threads) {
+        const int ct = threads / kg * rc;
         return (long long)a.n_seqs * a.H * ((a.e + ct - 1) / ct);
     };
-    if (blocks(256) >= tq_sm_count() / 2 && a.e >= 256 / KG * CS_RC) return launch_channel_scan<KG, RK, 256>(a, stream);
-    if (blocks(128) >= tq_sm_count() / 2 || KG == 8) return launch_channel_scan<KG, RK, 128>(a, stream);
-    return launch_channel_scan<KG, RK, 64>(a, stream);
+    if constexpr (RK == 4 && KG >= 16) {
+        constexpr int HALF = KG / 2;
+        if (blocks(HALF, 4, 128) > 2ll * tq_sm_count() && a.e >= 128 / HALF * 4)
+            return launch_channel_scan<HALF, 8, 4, 128>(a, stream);
+    }
+    if (blocks(KG, 2, 256) >= tq_sm_count() / 2 && a.e >= 256 / KG * 2) return launch_channel_scan<KG, RK, 2, 256>(a, stream);
+    if (blocks(KG, 2, 128) >= tq_sm_count() / 2 || KG == 8) return launch_channel_scan<KG, RK, 2, 128>(a, stream);
+    return launch_channel_scan<KG, RK, 2, 64>(a, stream);
 }
 
 // Floats of the records for a step of n_tokens tokens in n_seqs sequences, heads H of d keys.
