@@ -55,7 +55,7 @@ G_A = model(300, 96, 1e-6, 3, 0.8, 3.0, [
 G_B = model(384, 160, 1e-6, 2, 0.6, 2.0, [
     {**delta(4, 2, 64, 64, 4), "mlp": moe(96, 8, 2, (4, 2), shared=64)},
     {**both(4, 2, 64, 64, 128, 0.15, 160, 0.9, 0.6), "mlp": dense(256)},
-    {**both(2, 1, 128, 128, 65, 0.1, 96, 1.2, 0.8, base=50000.0), "mlp": moe(64, 8, 3, (2, 1))},
+    {**both(2, 1, 128, 128, 65, 0.1, 96, 1.2, 0.8, base=50000.0), "mlp": moe(64, 12, 3, (2, 1))},
     {**delta(4, 2, 64, 64, 4), "mlp": moe(96, 8, 2, (4, 2), shared=64), "weights_of": 0},
     {**delta(1, 1, 128, 128, 2), "mlp": None},
     {**both(4, 4, 32, 32, None, 0.2, 128, 1.0, 1.0, dims=16), "mlp": dense(96)},

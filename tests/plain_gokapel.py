@@ -171,7 +171,7 @@ def gru_scan(z, cand):
 
 
 def min_gru(x, w, p):
-    """A recurrence whose gates read the current token only: z = sigma(W_z x + b_z), u = W_x x + b_x, the candidate
+    """One number of memory per channel, an update gate that does not look at it: z = sigma(W_z x + b_z), u = W_x x + b_x, the candidate
     is u + 1/2 for u >= 0 and sigma(u) below; result W_o (S * silu(W_g x))."""
     z = torch.sigmoid(x @ w[p + "z"].T + w[p + "z.b"])
     u = x @ w[p + "x"].T + w[p + "x.b"]

@@ -1,4 +1,4 @@
-// A gated recurrence per channel whose gates read the current token only (minGRU):
+// A recurrence per channel with an update gate that does not look at the state (minGRU):
 //
 //   z = sigmoid(z~),  c = u + 1/2 for u >= 0, sigmoid(u) below      (z~, u: projections with their biases)
 //   S_t = (1 - z_t) S_{t-1} + z_t c_t                                per channel, S zero at first

@@ -1,4 +1,4 @@
-"""A mixer whose memory is one number per channel, with gates that read the current token only (minGRU):
+"""A mixer whose memory is one number per channel, with an update gate that does not look at it (minGRU):
 
     z = sigmoid(W_z x + b_z),   u = W_x x + b_x,   c = u + 1/2 for u >= 0, sigmoid(u) below
     S_t = (1 - z) S_{t-1} + z c                       entry by entry, `width` channels

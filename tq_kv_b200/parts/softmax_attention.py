@@ -115,7 +115,7 @@ class SoftmaxAttention(Mixer):
         if self.qk_norm_weights and not self.qk_norm_eps:
             raise ConfigError("softmax attention: qk_norm_weights belong to a norm per head (qk_norm_eps)")
         self.result_scale = float(p.get("result_scale", 1.0))
-        if self.result_scale != 1.0 and self.shared_kv_given(p):
+        if self.result_scale != 1.0 and (p.get("shared_kv") or p.get("shares_packed")):
             raise ConfigError("softmax attention: result_scale rides in the values, a layer that reads another's cache has none")
         self.shared_kv = bool(p.get("shared_kv", False))
         self.shares_packed = bool(p.get("shares_packed", False))
@@ -140,10 +140,6 @@ class SoftmaxAttention(Mixer):
         self.o_width = self.n_heads * self.value_dim
         self.w_in = self.w_o = self.slopes = self.sinks = None
         self.window_chunk = 1
-
-    @staticmethod
-    def shared_kv_given(p) -> bool:
-        return bool(p.get("shared_kv", False)) or bool(p.get("shares_packed", False))
 
     # ---- weights ----------------------------------------------------------
     def _n(self, which: str) -> str:
