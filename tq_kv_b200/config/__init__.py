@@ -17,6 +17,9 @@ from .registry import (Architecture, register_architecture, registered_architect
 from .rirudra import ARCHITECTURE as RIRUDRA_ARCHITECTURE
 from .rirudra import MODEL_TYPE as RIRUDRA_MODEL_TYPE
 from .rirudra import RirudraConfig, build_rirudra_spec
+from .safurax import ARCHITECTURE as SAFURAX_ARCHITECTURE
+from .safurax import MODEL_TYPE as SAFURAX_MODEL_TYPE
+from .safurax import SafuraxConfig, build_safurax_spec
 from .shapes import named_shape, shape_names
 from .zodosun import ARCHITECTURE as ZODOSUN_ARCHITECTURE
 from .zodosun import MODEL_TYPE as ZODOSUN_MODEL_TYPE
@@ -40,7 +43,11 @@ register_architecture(
 register_architecture(
     Architecture(GOKAPEL_ARCHITECTURE, GOKAPEL_MODEL_TYPE, GokapelConfig, build_gokapel_spec), replace=True)
 
+register_architecture(
+    Architecture(SAFURAX_ARCHITECTURE, SAFURAX_MODEL_TYPE, SafuraxConfig, build_safurax_spec), replace=True)
+
 __all__ = [
+    "SafuraxConfig", "build_safurax_spec",
     "GokapelConfig", "build_gokapel_spec",
     "FuresunConfig", "build_furesun_spec",
     "PavisunConfig", "build_pavisun_spec",

@@ -146,7 +146,7 @@ __global__ void attention_kernel(const TC* __restrict__ q, KVSource src, const i
             }
         }
 
-        if (n_splits == 1) {
+        if (!part_acc) {
             if (opt.sinks) {                                 // the sink's exp(sink - m), the maximum moved up to it
                 const float sink = opt.sinks[h];
                 const float m_new = fmaxf(m, sink);
@@ -213,7 +213,8 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_acc, const
     }
 }
 
-// Scratch needed for n_splits > 1: part_acc float[T*nh*n_splits*vd], part_ml float[T*nh*n_splits*2].
+// Scratch needed for n_splits > 1: part_acc float[T*nh*n_splits*vd], part_ml float[T*nh*n_splits*2].  Without `out`
+// the parts are what the caller wants (one per split, of one split too; no sink then): nothing is merged.
 // hd and vd: multiples of 8 up to 512 (rows of the cache then start on 16-byte boundaries in either precision).
 TQ_API int tq_attention_ext(const void* q, int dtype, const void* k_packed, const void* v_packed, const void* k_pages,
                             const void* v_pages, const int* block_table, int table_width, int ring_pages,
@@ -225,7 +226,8 @@ TQ_API int tq_attention_ext(const void* q, int dtype, const void* k_packed, cons
     if (hd <= 0 || hd > 64 * ATT_MAX_PAIRS || hd % 8 || nkv <= 0 || nh % nkv) return (int)cudaErrorInvalidValue;
     if (vd <= 0 || vd > 64 * ATT_MAX_PAIRS || vd % 8 || keep_first < 0) return (int)cudaErrorInvalidValue;
     if (keep_first > 0 && ring_pages > 0) return (int)cudaErrorInvalidValue;   // a ring has overwritten them
-    if (n_splits < 1 || (n_splits > 1 && (!part_acc || !part_ml))) return (int)cudaErrorInvalidValue;
+    if (n_splits < 1 || ((n_splits > 1 || !out) && (!part_acc || !part_ml)) || (!out && sinks)) return (int)cudaErrorInvalidValue;
+    if (n_splits == 1 && out) part_acc = part_ml = nullptr;
     if (!k_packed && (!k_pages || !block_table || page_tokens <= 0)) return (int)cudaErrorInvalidValue;
     if (nkv > 65535 || n_splits > 65535) return (int)cudaErrorInvalidValue;
     KVSource src{k_packed, v_packed, k_pages, v_pages, block_table, table_width, ring_pages, page_tokens};
@@ -246,7 +248,7 @@ TQ_API int tq_attention_ext(const void* q, int dtype, const void* k_packed, cons
     else
         return (int)cudaErrorInvalidValue;
     int st = tq_launch_status();
-    if (st || n_splits == 1) return st;
+    if (st || !part_acc || !out) return st;
     const dim3 mgrid(n_tokens, nh);
     if (dtype == TQ_F32)
         attention_merge_kernel<float><<<mgrid, 128, 0, stream>>>(part_acc, part_ml, (float*)out, nh, vd, n_splits, sinks);

@@ -1,5 +1,5 @@
-// Memory-bound kernels around the matrix products: embedding gather, RMS
-// norm, bias + rotary position encoding + cache append, SwiGLU gating.
+// Memory-bound kernels around the matrix products: embedding gather, RMS and
+// layer norm, bias + rotary position encoding + cache append, SwiGLU gating.
 // All arithmetic is float32; T* parameters are float or bfloat16.
 #include "common.cuh"
 
@@ -49,8 +49,10 @@ TQ_API int tq_embed(const int* tokens, const void* table, int table_dtype, float
 // (src/models/turbo_generic.rs:41-51).  x is the float32 residual stream;
 // `rows` (optional) selects the input rows, so that the final norm touches
 // only the rows whose logits are wanted.
+// CENTER: the layer norm, y = c / sqrt(mean(c^2) + eps) * w with c = x - mean(x): the mean is taken first and the
+// deviations' squares are summed, not the difference of two large sums.
 // ---------------------------------------------------------------------------
-template <typename TO>
+template <typename TO, bool CENTER>
 __global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, TO* __restrict__ out,
                                const int* __restrict__ rows, int H, float eps) {
     __shared__ float red[32];
@@ -59,37 +61,45 @@ __global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restr
     pdl_launch();
     const float* xr = x + (size_t)(rows ? rows[r] : r) * H;
     TO* o = out + (size_t)r * H;
-    float ss = 0.f;
+    float ss = 0.f, mean = 0.f;
+    if constexpr (CENTER) {
+        float sum = 0.f;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) sum += xr[i];
+        mean = block_sum(sum, red) / (float)H;
+    }
     if ((H & 3) == 0) {                       // rows are 16-byte aligned: four values per load
         const float4* x4 = reinterpret_cast<const float4*>(xr);
         const float4* w4 = reinterpret_cast<const float4*>(w);
         for (int i = threadIdx.x; i < (H >> 2); i += blockDim.x) {
-            const float4 v = x4[i];
+            float4 v = x4[i];
+            if (CENTER) { v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean; }
             ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
         }
         ss = block_sum(ss, red);
         const float rms = sqrtf(ss / (float)H + eps);
         for (int i = threadIdx.x; i < (H >> 2); i += blockDim.x) {
-            const float4 v = x4[i], g = w4[i];
+            float4 v = x4[i];
+            const float4 g = w4[i];
+            if (CENTER) { v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean; }
             store2_f32<TO>(o + 4 * i, (v.x / rms) * g.x, (v.y / rms) * g.y);
             store2_f32<TO>(o + 4 * i + 2, (v.z / rms) * g.z, (v.w / rms) * g.w);
         }
         return;
     }
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float v = xr[i];
+        const float v = xr[i] - mean;
         ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, red);
     const float rms = sqrtf(ss / (float)H + eps);
-    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = from_f32<TO>((xr[i] / rms) * w[i]);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = from_f32<TO>(((xr[i] - mean) / rms) * w[i]);
 }
 
 // Rows of up to 8,192 values in steps of four: a row is read once and held in registers between the sum of
 // squares and the scaling (VPT 16-byte loads per thread, all in flight together, the norm's weights with them).
 // A prompt's many rows get small blocks, so that a whole wave of rows is resident; the few rows of a decode
 // step get wide ones, so that a row is one round of loads.  Same arithmetic as above.
-template <typename TO, int THREADS, int VPT>
+template <typename TO, int THREADS, int VPT, bool CENTER>
 __global__ void __launch_bounds__(THREADS)
 rmsnorm_cached_kernel(const float* __restrict__ x, const float* __restrict__ w, TO* __restrict__ out,
                       const int* __restrict__ rows, int H, float eps) {
@@ -112,6 +122,15 @@ rmsnorm_cached_kernel(const float* __restrict__ x, const float* __restrict__ w, 
         const int idx = threadIdx.x + i * THREADS;
         v[i] = idx < h4 ? x4[idx] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    if constexpr (CENTER) {
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+        const float mean = block_sum(sum, red) / (float)H;
+#pragma unroll
+        for (int i = 0; i < VPT; ++i)
+            if (threadIdx.x + i * THREADS < h4) { v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean; }
+    }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
         ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
@@ -129,12 +148,12 @@ rmsnorm_cached_kernel(const float* __restrict__ x, const float* __restrict__ w, 
     }
 }
 
-template <typename TO>
+template <typename TO, bool CENTER>
 static int launch_rmsnorm_cached(const float* x, const float* w, TO* out, const int* rows, int n_rows, int H, float eps,
                                  cudaStream_t stream) {
     const int h4 = H >> 2;
 #define TQ_RN(T, V)                                                                                                 \
-    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, rmsnorm_cached_kernel<TO, T, V>, dim3(n_rows), dim3(T), 0, stream, x, w, \
+    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, rmsnorm_cached_kernel<TO, T, V, CENTER>, dim3(n_rows), dim3(T), 0, stream, x, w, \
                          out, rows, H, eps)
     if (n_rows < 128) {                                    // a decode step: wide blocks
         if (h4 <= 128) TQ_RN(128, 1);
@@ -149,21 +168,33 @@ static int launch_rmsnorm_cached(const float* x, const float* w, TO* out, const 
 #undef TQ_RN
 }
 
-TQ_API int tq_rmsnorm(const float* x, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int H,
-                      float eps, cudaStream_t stream) {
+template <bool CENTER>
+static int launch_rmsnorm(const float* x, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int H,
+                          float eps, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if ((H & 3) == 0 && H <= 256 * 8 * 4 && (out_dtype == TQ_F32 || out_dtype == TQ_BF16)) {
-        if (out_dtype == TQ_F32) return launch_rmsnorm_cached<float>(x, w, (float*)out, rows, n_rows, H, eps, stream);
-        return launch_rmsnorm_cached<bf16>(x, w, (bf16*)out, rows, n_rows, H, eps, stream);
+        if (out_dtype == TQ_F32)
+            return launch_rmsnorm_cached<float, CENTER>(x, w, (float*)out, rows, n_rows, H, eps, stream);
+        return launch_rmsnorm_cached<bf16, CENTER>(x, w, (bf16*)out, rows, n_rows, H, eps, stream);
     }
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     if (out_dtype == TQ_F32)
-        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, x, w, (float*)out, rows,
-                             H, eps);
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, rmsnorm_kernel<float, CENTER>, dim3(n_rows), dim3(threads), 0, stream, x, w,
+                             (float*)out, rows, H, eps);
     if (out_dtype == TQ_BF16)
-        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, rmsnorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, x, w, (bf16*)out, rows, H,
-                             eps);
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, rmsnorm_kernel<bf16, CENTER>, dim3(n_rows), dim3(threads), 0, stream, x, w,
+                             (bf16*)out, rows, H, eps);
     return (int)cudaErrorInvalidValue;
+}
+
+TQ_API int tq_rmsnorm(const float* x, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int H,
+                      float eps, cudaStream_t stream) {
+    return launch_rmsnorm<false>(x, w, out, out_dtype, rows, n_rows, H, eps, stream);
+}
+
+TQ_API int tq_layernorm(const float* x, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int H,
+                        float eps, cudaStream_t stream) {
+    return launch_rmsnorm<true>(x, w, out, out_dtype, rows, n_rows, H, eps, stream);
 }
 
 // ---------------------------------------------------------------------------

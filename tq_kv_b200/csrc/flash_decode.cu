@@ -354,7 +354,7 @@ flash_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
             }
         }
         const int h = g * n_rep + r;
-        if (n_splits == 1) {
+        if (n_splits == 1 && out) {
             if (WEIGHTS == FD_SOFTMAX_EXT && opt.sinks) {     // (with splits the merge step adds the sink)
                 const float sink = opt.sinks[h] * 1.4426950408889634f;
                 const float m2 = fmaxf(m, sink), f = exp2f(m - m2);
@@ -480,7 +480,8 @@ TQ_API int tq_sigmoid_flash_decode(const void* q, const void* k_pages, const voi
 
 
 // The softmax kernel with options (FD_SOFTMAX_EXT above): keys and values of one width.  Kept first tokens need a
-// cache that keeps all keys (no ring).  Returns cudaErrorNotSupported (801) for shapes outside this kernel's reach.
+// cache that keeps all keys (no ring).  k_pages == v_pages: the values are the keys.  Without `out` the parts are what
+// the caller wants (one per split, of one split too; no sink then).  Returns cudaErrorNotSupported (801) for shapes outside this kernel's reach.
 TQ_API int tq_flash_decode_ext(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                int table_width, int ring_pages, int page_tokens, const int* tok_pos, const int* tok_seq,
                                int window, float scale, float softcap, const float* slopes, int keep_first,
@@ -495,16 +496,16 @@ TQ_API int tq_flash_decode_ext(const void* q, const void* k_pages, const void* v
     if (kv_div > 64) return (int)cudaErrorNotSupported;
     nkv *= kv_div;
     if (nkv > 65535 || n_splits > 65535) return (int)cudaErrorNotSupported;
-    if (n_splits < 1 || (n_splits > 1 && (!part_acc || !part_ml))) return (int)cudaErrorInvalidValue;
+    if (n_splits < 1 || ((n_splits > 1 || !out) && (!part_acc || !part_ml)) || (!out && sinks)) return (int)cudaErrorInvalidValue;
     if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
     const FdOptions opt{scale, softcap, slopes, window > 0 ? keep_first : 0, sinks, chunk};
-#define TQ_FD(H)                                                                                                        \
-    case H:                                                                                                             \
-        return launch_flash_decode<H, FD_SOFTMAX_EXT>((const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages,      \
-                                                      block_table, table_width, ring_pages, tok_pos, tok_seq, window,   \
-                                                      scale, (bf16*)out, part_acc, part_ml, n_tokens, nh, nkv,          \
-                                                      n_splits, TQ_PDL_FLASH_DECODE, stream, nullptr, 0, nullptr, 0,    \
-                                                      kv_div, opt)
+    const bool same = k_pages == v_pages;
+#define TQ_FD_ARGS (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, block_table, table_width, ring_pages,      \
+                   tok_pos, tok_seq, window, scale, (bf16*)out, part_acc, part_ml, n_tokens, nh, nkv, n_splits,            \
+                   TQ_PDL_FLASH_DECODE, stream, nullptr, 0, nullptr, 0, kv_div, opt
+#define TQ_FD(H)                                                                                                      \
+    case H:                                                                                                           \
+        return same ? launch_flash_decode<H, FD_SOFTMAX_EXT, 0>(TQ_FD_ARGS) : launch_flash_decode<H, FD_SOFTMAX_EXT, 1>(TQ_FD_ARGS)
     switch (hd) {
         TQ_FD(32);
         TQ_FD(64);
@@ -512,5 +513,6 @@ TQ_API int tq_flash_decode_ext(const void* q, const void* k_pages, const void* v
         TQ_FD(128);
         default: return (int)cudaErrorNotSupported;
     }
+#undef TQ_FD_ARGS
 #undef TQ_FD
 }

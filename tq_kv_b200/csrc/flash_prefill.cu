@@ -67,6 +67,7 @@ struct FpOptions {
     int ldg;
     const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
     int chunk;              // > 0: keys of the query's own chunk only
+    float* out32;           // the result goes here unrounded, [T, nh * HD] (`out` is then not used); or null
 };
 
 // cap * tanh(x / cap) with 2^x and a fast division (a few ulp; tanh.approx is not enough)
@@ -302,7 +303,10 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
                 a = __fdividef(a, 1.f + __expf(-grow[d]));
                 c = __fdividef(c, 1.f + __expf(-grow[d + 1]));
             }
-            *reinterpret_cast<__nv_bfloat162*>(orow + d) = __floats2bfloat162_rn(a, c);
+            if (EXT && opt.out32)
+                *reinterpret_cast<float2*>(opt.out32 + ((size_t)(tok0 + ri[r]) * nh + h) * HD + d) = make_float2(a, c);
+            else
+                *reinterpret_cast<__nv_bfloat162*>(orow + d) = __floats2bfloat162_rn(a, c);
         }
     }
 }
@@ -310,7 +314,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
 template <int HD, bool EXT = false>
 static int launch_flash_prefill(const bf16* q, const FpSource& src, const int* cu_seqlens, const int* start_pos,
                                 int n_seqs, int n_tokens, int window, float scale, bf16* out, int nh, int nkv,
-                                cudaStream_t stream, FpOptions opt = FpOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0}) {
+                                cudaStream_t stream, FpOptions opt = FpOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0, nullptr}) {
     constexpr size_t smem = 2 * 2 * FP_BN * (HD * 2 + 16);
     static bool configured = false;
     if (!configured) {
@@ -358,8 +362,8 @@ TQ_API int tq_flash_prefill_ext(const void* q, const void* k_packed, const void*
                                 const void* v_pages, const int* block_table, int table_width, int ring_pages,
                                 int page_tokens, const int* cu_seqlens, const int* start_pos, int n_seqs, int n_tokens,
                                 int window, float scale, float softcap, const float* slopes, int keep_first,
-                                const float* sinks, int chunk, const float* gate, int ldg, void* out, int nh, int nkv, int hd,
-                                cudaStream_t stream) {
+                                const float* sinks, int chunk, const float* gate, int ldg, void* out, int out_f32, int nh,
+                                int nkv, int hd, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (nkv <= 0 || nh % nkv || nh > 65535) return (int)cudaErrorNotSupported;
     if (!k_packed && (!k_pages || !block_table || page_tokens <= 0)) return (int)cudaErrorInvalidValue;
@@ -367,7 +371,7 @@ TQ_API int tq_flash_prefill_ext(const void* q, const void* k_packed, const void*
     FpSource src{(const bf16*)k_packed, (const bf16*)v_packed, (const bf16*)k_pages, (const bf16*)v_pages,
                  block_table, table_width, ring_pages, page_tokens};
     if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
-    const FpOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk};
+    const FpOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk, out_f32 ? (float*)out : nullptr};
 #define TQ_FP(H)                                                                                                    \
     case H:                                                                                                         \
         return launch_flash_prefill<H, true>((const bf16*)q, src, cu_seqlens, start_pos, n_seqs, n_tokens, window, \

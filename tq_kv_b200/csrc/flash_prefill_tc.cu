@@ -175,6 +175,7 @@ struct FtOptions {
     int ldg;
     const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
     int chunk;              // > 0: keys of the query's own chunk only
+    float* out32;           // the result goes here unrounded, [T, nh * HD] (`out` is then not used); or null
 };
 
 template <int HD, bool PAGED, int WEIGHTS>
@@ -546,7 +547,15 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                         v[d + 3] = __fdividef(v[d + 3], 1.f + __expf(-gv.w));
                     }
                 }
-                if (i_row < len) {
+                if (WEIGHTS == FT_SOFTMAX_EXT && opt.out32) {
+                    if (i_row < len) {
+                        float* o32 = opt.out32 + ((size_t)(tok0 + i_row) * nh + h) * HD + c;
+#pragma unroll
+                        for (int d = 0; d < 32; d += 4)
+                            *reinterpret_cast<float4*>(o32 + d) =
+                                make_float4(v[d] * inv, v[d + 1] * inv, v[d + 2] * inv, v[d + 3] * inv);
+                    }
+                } else if (i_row < len) {
 #pragma unroll
                     for (int d = 0; d < 32; d += 8) {
                         __nv_bfloat162 a = __floats2bfloat162_rn(v[d] * inv, v[d + 1] * inv);
@@ -586,7 +595,7 @@ static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
                      int table_width, int ring_pages, const int* cu_seqlens, const int* start_pos, int n_seqs,
                      int n_tokens, int window, float scale, bf16* out, int nh, int nkv, int* status,
                      cudaStream_t stream, const float* bias = nullptr, int n_dist = 0, const float* gate = nullptr,
-                     int ldg = 0, FtOptions opt = FtOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0}) {
+                     int ldg = 0, FtOptions opt = FtOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0, nullptr}) {
     constexpr int SMEM = (HD / 64) * (FT_SUB_BYTES + 4 * FT_KV_SUB_BYTES) + 256;
     static bool configured = false;
     if (!configured) {
@@ -679,7 +688,7 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
                                    int ring_pages, int page_tokens, const int* cu_seqlens, const int* start_pos,
                                    int n_seqs, int n_tokens, int window, float scale, float softcap,
                                    const float* slopes, int keep_first, const float* sinks, int chunk,
-                                   const float* gate, int ldg, void* out, int nh,
+                                   const float* gate, int ldg, void* out, int out_f32, int nh,
                                    int nkv, int hd, int* status, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (nkv <= 0 || nh % nkv || (hd != 64 && hd != 128)) return (int)cudaErrorNotSupported;
@@ -700,7 +709,7 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
     }
     if (st) return st;
     if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
-    const FtOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk};
+    const FtOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk, out_f32 ? (float*)out : nullptr};
 #define TQ_FT(H, P) return ft_launch<H, P, FT_SOFTMAX_EXT>(mq, mk, mv, block_table, table_width, ring_pages, cu_seqlens, \
                                                            start_pos, n_seqs, n_tokens, window, scale, (bf16*)out, nh,    \
                                                            nkv, status, stream, nullptr, 0, nullptr, 0, opt)

@@ -13,7 +13,8 @@
 //                  packed rows and / or the sequence's page; rows are padded with zeros to the width `rp` the
 //                  attention kernels take
 //   latent_query   per (token, head): q~ as above
-//   latent_expand  per (token, head): o[h] = U_v[h] mean(c), times sigmoid(gate) entry by entry
+//   latent_expand  per (token, head): o[h] = U_v[h] mean(c), times sigmoid(gate) entry by entry or (head_gate) with one
+//                  gate per head
 //
 //   latent_heads   for prompts that bring all their keys along: per (token, head) the query [q_flat, rot(q_rot), 0 ...],
 //                  the expanded key [U_k[h] c, k_r, 0 ...] and the value [U_v[h] c, 0 ...], all `hw` wide, for the
@@ -149,7 +150,7 @@ __global__ void latent_heads_kernel(const float* __restrict__ q, int ldq, const 
 
 template <typename T>
 __global__ void latent_expand_kernel(const T* __restrict__ lat, int H, int n, int rp, int e, const T* __restrict__ uv,
-                                     const float* __restrict__ gate, int ldg, T* __restrict__ out) {
+                                     const float* __restrict__ gate, int ldg, int head_gate, T* __restrict__ out) {
     extern __shared__ float sh[];          // [n] the head's mean latent
     const int t = blockIdx.x, h = blockIdx.y;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
@@ -162,7 +163,7 @@ __global__ void latent_expand_kernel(const T* __restrict__ lat, int H, int n, in
         for (int j = threadIdx.x; j < e; j += blockDim.x) {
             const size_t c = (size_t)h * e + j;
             float acc = sh[j];
-            if (gate) acc *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + c]));
+            if (gate) acc *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + (head_gate ? h : c)]));
             out[(size_t)t * H * e + c] = from_f32<T>(acc);
         }
         return;
@@ -174,7 +175,7 @@ __global__ void latent_expand_kernel(const T* __restrict__ lat, int H, int n, in
         acc = warp_sum(acc);
         if (lane == 0) {
             const size_t c = (size_t)h * e + j;
-            if (gate) acc *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + c]));
+            if (gate) acc *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + (head_gate ? h : c)]));
             out[(size_t)t * H * e + c] = from_f32<T>(acc);
         }
     }
@@ -225,17 +226,17 @@ TQ_API int tq_latent_query(const float* q, int ldq, int H, int d, int r, int n, 
 }
 
 TQ_API int tq_latent_expand(const void* lat, int H, int n, int rp, int e, const void* uv, const float* gate, int ldg,
-                            void* out, int dtype, int n_tokens, cudaStream_t stream) {
+                            int head_gate, void* out, int dtype, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (!lat || !out || H <= 0 || H > 65535 || n <= 0 || rp < n || e <= 0 || (!uv && e > n)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)n * sizeof(float);
     const dim3 grid(n_tokens, H);
     if (dtype == TQ_F32)
         return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_expand_kernel<float>, grid, dim3(128), smem, stream,
-                             (const float*)lat, H, n, rp, e, (const float*)uv, gate, ldg, (float*)out);
+                             (const float*)lat, H, n, rp, e, (const float*)uv, gate, ldg, head_gate, (float*)out);
     if (dtype == TQ_BF16)
         return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_expand_kernel<bf16>, grid, dim3(128), smem, stream,
-                             (const bf16*)lat, H, n, rp, e, (const bf16*)uv, gate, ldg, (bf16*)out);
+                             (const bf16*)lat, H, n, rp, e, (const bf16*)uv, gate, ldg, head_gate, (bf16*)out);
     return (int)cudaErrorInvalidValue;
 }
 

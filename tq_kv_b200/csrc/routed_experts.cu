@@ -40,19 +40,20 @@ TQ_API int tq_table_choice(const int* tokens, const int* table, int vocab, int t
 }
 
 // ---- choice: experts of each token from a router's logits -------------------------------------------------------
-// scores s = sigmoid(logit); the `top` largest are chosen (the lowest index first among equals); their weights
-// are  scale * s / (sum of the chosen s + floor).  The choice compares the logits themselves: the sigmoid keeps
+// scores s = sigmoid(logit), or with softmax != 0 s = exp(logit); the `top` largest are chosen (the lowest index first
+// among equals); their weights are  scale * s / (sum of the chosen s + floor): with softmax (floor 0 and scale 1) the
+// softmax over the chosen logits, taken relative to the largest, which is chosen first.  The choice compares the logits themselves: the sigmoid keeps
 // their order, but in float32 it is 1 for every logit above 17 and would make equals of them.  A warp per token;
 // float32 throughout.
 __global__ void __launch_bounds__(128)
 router_choice_kernel(const float* __restrict__ logits, int ld, int n_experts, int top, float scale, float floor_,
-                     int* __restrict__ choice, float* __restrict__ weights, int n_tokens) {
+                     int softmax, int* __restrict__ choice, float* __restrict__ weights, int n_tokens) {
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= n_tokens) return;
     pdl_wait();
     pdl_launch();
     const float* z = logits + (size_t)t * ld;
-    float total = 0.f;
+    float total = 0.f, first = 0.f;
     for (int s = 0; s < top; ++s) {
         float best = 0.f;
         int best_e = n_experts;                           // n_experts: this lane has found none yet
@@ -68,7 +69,9 @@ router_choice_kernel(const float* __restrict__ logits, int ld, int n_experts, in
             const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
             if (oe < n_experts && (best_e == n_experts || ob > best || (ob == best && oe < best_e))) { best = ob; best_e = oe; }
         }
-        const float score = 1.f / (1.f + expf(-best));
+        if (s == 0) first = best;
+        if (best_e >= n_experts) best_e = 0;              // (logits that are no numbers choose nothing)
+        const float score = softmax ? expf(best - first) : 1.f / (1.f + expf(-best));
         if (lane == 0) { choice[t * top + s] = best_e; weights[t * top + s] = score; }
         __syncwarp();
         total += score;
@@ -77,12 +80,12 @@ router_choice_kernel(const float* __restrict__ logits, int ld, int n_experts, in
     for (int s = lane; s < top; s += 32) weights[t * top + s] *= f;
 }
 
-TQ_API int tq_router_choice(const float* logits, int ld, int n_experts, int top, float scale, float floor_, int* choice,
-                            float* weights, int n_tokens, cudaStream_t stream) {
+TQ_API int tq_router_choice(const float* logits, int ld, int n_experts, int top, float scale, float floor_, int softmax,
+                            int* choice, float* weights, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (!logits || !choice || !weights || top < 1 || top > n_experts) return (int)cudaErrorInvalidValue;
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, router_choice_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, stream, logits,
-                         ld, n_experts, top, scale, floor_, choice, weights, n_tokens);
+                         ld, n_experts, top, scale, floor_, softmax, choice, weights, n_tokens);
 }
 
 // ---- choice with groups --------------------------------------------------------------------------------------
@@ -229,7 +232,7 @@ template <typename TA, typename TW>
 __global__ void __launch_bounds__(256)
 routed_down_kernel(const TA* __restrict__ act, const TW* __restrict__ w_down, const int* __restrict__ choice,
                    const float* __restrict__ weights, int top, int W, int F, float* __restrict__ y, int accumulate,
-                   bool vec) {
+                   bool vec, const float* __restrict__ shared, const float* __restrict__ shared_gate, int ldg) {
     const int t = blockIdx.x;
     const int c = blockIdx.y * 8 + (threadIdx.x >> 5);
     if (c >= W) return;
@@ -243,7 +246,8 @@ routed_down_kernel(const TA* __restrict__ act, const TW* __restrict__ w_down, co
     }
     if ((threadIdx.x & 31) == 0) {
         float* o = y + (size_t)t * W + c;
-        const float v = weights ? sum : sum / (float)top;
+        float v = weights ? sum : sum / (float)top;
+        if (shared) v += shared[(size_t)t * W + c] / (1.f + expf(-shared_gate[(size_t)t * ldg]));
         *o = accumulate ? *o + v : v;
     }
 }
@@ -251,11 +255,14 @@ routed_down_kernel(const TA* __restrict__ act, const TW* __restrict__ w_down, co
 static inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 // x [T, W] (row stride ldx), act [T*top, F] of x's dtype (scratch), y [T, W] float32.  Weights float32 or bfloat16.
-// gated 0: experts without a gate, w_gu [E, F, W].
+// gated 0: experts without a gate, w_gu [E, F, W].  shared (or null): float32 [T, W], another result of every token,
+// added times sigmoid(shared_gate[t * ldg]).
 TQ_API int tq_routed_experts_rows(const void* x, int x_dtype, int ldx, const void* w_gu, const void* w_down, int w_dtype,
                                   const int* choice, const float* weights, int top, int n_tokens, int W, int F,
-                                  void* act, float* y, int accumulate, int gated, cudaStream_t stream) {
+                                  void* act, float* y, int accumulate, int gated, const float* shared,
+                                  const float* shared_gate, int ldg, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (shared && !shared_gate) return (int)cudaErrorInvalidValue;
     if (top < 1 || W <= 0 || F <= 0) return (int)cudaErrorInvalidValue;
     const int xs = x_dtype == TQ_BF16 ? 2 : 4, ws = w_dtype == TQ_BF16 ? 2 : 4;
     const bool vec_up = W % 8 == 0 && aligned16(x) && aligned16(w_gu) && ((size_t)ldx * xs) % 16 == 0;
@@ -271,7 +278,7 @@ TQ_API int tq_routed_experts_rows(const void* x, int x_dtype, int ldx, const voi
                                (const TX*)x, ldx, (const TW*)w_gu, choice, top, W, F, (TX*)act, vec_up);             \
     if (st) return st;                                                                                                \
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, routed_down_kernel<TX, TW>, g2, dim3(256), 0, stream, (const TX*)act,   \
-                         (const TW*)w_down, choice, weights, top, W, F, y, accumulate, vec_down)
+                         (const TW*)w_down, choice, weights, top, W, F, y, accumulate, vec_down, shared, shared_gate, ldg)
     if (x_dtype == TQ_F32 && w_dtype == TQ_F32) { TQ_RUN(float, float); }
     if (x_dtype == TQ_F32 && w_dtype == TQ_BF16) { TQ_RUN(float, bf16); }
     if (x_dtype == TQ_BF16 && w_dtype == TQ_BF16) { TQ_RUN(bf16, bf16); }
@@ -330,10 +337,12 @@ routed_gather_kernel(const bf16* __restrict__ x, int ldx, const int* __restrict_
     for (int d = lane; d < W / 8; d += 32) dst[d] = src[d];
 }
 
-// y[t] (=, +=) 1/top * sum_s out[pos[t*top + s]] (the experts in the table's order): float32, W % 4 == 0
+// y[t] (=, +=) 1/top * sum_s out[pos[t*top + s]] (the experts in the table's order) [+ sigmoid(shared_gate[t]) *
+// shared[t]]: float32, W % 4 == 0
 __global__ void __launch_bounds__(256)
 routed_combine_kernel(const float* __restrict__ out, const int* __restrict__ pos, const float* __restrict__ weights,
-                      int top, int W, int n_tokens, float* __restrict__ y, int accumulate) {
+                      int top, int W, int n_tokens, float* __restrict__ y, int accumulate, const float* __restrict__ shared,
+                      const float* __restrict__ shared_gate, int ldg) {
     pdl_wait();
     pdl_launch();
     const int per_row = W / 4;
@@ -345,6 +354,11 @@ routed_combine_kernel(const float* __restrict__ out, const int* __restrict__ pos
         for (int s = 0; s < top; ++s) {
             const float4 v = reinterpret_cast<const float4*>(out + (size_t)pos[t * top + s] * W)[c];
             const float ws = weights ? weights[t * top + s] : 1.f;
+            a.x = fmaf(ws, v.x, a.x); a.y = fmaf(ws, v.y, a.y); a.z = fmaf(ws, v.z, a.z); a.w = fmaf(ws, v.w, a.w);
+        }
+        if (shared) {                                     // (then there are weights: inv is 1)
+            const float4 v = reinterpret_cast<const float4*>(shared + (size_t)t * W)[c];
+            const float ws = 1.f / (1.f + expf(-shared_gate[(size_t)t * ldg]));
             a.x = fmaf(ws, v.x, a.x); a.y = fmaf(ws, v.y, a.y); a.z = fmaf(ws, v.z, a.z); a.w = fmaf(ws, v.w, a.w);
         }
         float4* o = reinterpret_cast<float4*>(y + (size_t)t * W) + c;
@@ -376,11 +390,13 @@ TQ_API int tq_routed_sort(const void* x, int ldx, const int* choice, int top, in
 }
 
 TQ_API int tq_routed_combine(const float* out, const int* pos, const float* weights, int top, int n_tokens, int W,
-                             float* y, int accumulate, cudaStream_t stream) {
+                             float* y, int accumulate, const float* shared, const float* shared_gate, int ldg,
+                             cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (W % 4 || !aligned16(out) || !aligned16(y)) return (int)cudaErrorInvalidValue;
+    if (shared && (!shared_gate || !weights || !aligned16(shared))) return (int)cudaErrorInvalidValue;
     size_t blocks = ((size_t)n_tokens * (W / 4) + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     return tq_launch_pdl(TQ_PDL_ELEMENTWISE, routed_combine_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, out, pos,
-                         weights, top, W, n_tokens, y, accumulate);
+                         weights, top, W, n_tokens, y, accumulate, shared, shared_gate, ldg);
 }

@@ -10,6 +10,7 @@ from ._lib import KernelError, check, core, dtype_code, need_contiguous, ptr, st
 
 MAX_HEAD_DIM = 512    # of the general kernel; the Qwen2 configuration keeps its own limit of 256
 NOT_SUPPORTED = 801     # cudaErrorNotSupported: a specialised kernel declines the shape
+TENSOR_CORE_WIDTHS = (32, 64, 96, 128)      # head widths (keys and values alike) of the bfloat16 tensor-core kernels
 USE_TC_ATTENTION = True  # prompts: the tcgen05 kernel (csrc/flash_prefill_tc.cu) before the mma.sync one
 
 
@@ -135,7 +136,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
                   block_table: Optional[torch.Tensor] = None, table_width: int = 0, ring_pages: int = 0,
                   page_tokens: int = 64, n_splits: int = 1, scratch: Optional[torch.Tensor] = None,
                   gate: Optional[torch.Tensor] = None, use_fast: bool = True, sink=False,
-                  chunk: Optional[int] = None):
+                  chunk: Optional[int] = None, unmerged: bool = False):
     """Softmax attention with options: for the query at position i of head h and the key at position j <= i,
 
         s = q . k * scale;   s <- softcap * tanh(s / softcap)  (if a cap is given);
@@ -147,13 +148,19 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
     Value rows may have another width than the keys.  q [T, nh*key_dim], out [T, nh*value_dim]; keys and values as in `attention`.
     `gate` (float32 [T, nh*value_dim], possibly a column slice of wider rows): out *= sigmoid(gate), in the
     attention kernel's last step where it can, else by a kernel of its own.
+    `unmerged` (then `out` is None; no gate, no sink): the float32 results are returned for a kernel that goes on with
+    them, (rows [T, nh, value_dim], None, 1) or, per split of the keys, (sums [T, nh, n, value_dim], their maxima and
+    sums of weights [T, nh, n, 2], n), as `difference_of_maps` takes them.
 
     bfloat16 with keys and values of one width runs on the tensor cores: prompts on the tcgen05 kernel (heads of
     64 and 128) or the mma.sync one (32, 64, 96, 128), single tokens on the bandwidth-built cache kernel; all
     else, and float32, on the general kernel."""
     check_row_widths(n_heads, n_kv_heads, key_dim, value_dim)
     T = q.shape[0]
-    if q.shape[1] != n_heads * key_dim or tuple(out.shape) != (T, n_heads * value_dim) or out.dtype != q.dtype:
+    if unmerged and (out is not None or gate is not None or sink is not False):
+        raise KernelError("attention: unmerged results take no out, gate or sink")
+    if q.shape[1] != n_heads * key_dim or (not unmerged and (tuple(out.shape) != (T, n_heads * value_dim)
+                                                             or out.dtype != q.dtype)):
         raise KernelError("attention: q must be [T, n_heads*key_dim] and out [T, n_heads*value_dim] of one dtype")
     packed = k_packed is not None
     if packed:
@@ -179,8 +186,10 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
     if sink is not None and (sink.dtype != torch.float32 or tuple(sink.shape) != (n_heads,)):
         raise KernelError("attention: sink must be float32 [n_heads]")
     part_acc = part_ml = None
-    if n_splits > 1:
-        need = split_scratch_floats(T, n_heads, value_dim, n_splits)
+    if n_splits > 1 or unmerged:
+        need = T * n_heads * n_splits * (value_dim + 2)
+        if unmerged and scratch is None:
+            scratch = torch.empty(need, dtype=torch.float32, device=q.device)
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention: {n_splits} splits need {need} float32 of scratch")
         n_acc = T * n_heads * n_splits * value_dim
@@ -202,19 +211,21 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
                 ptr(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages),
                 0 if k_pages is None else k_pages.shape[0], ptr(block_table), table_width, ring_pages, page_tokens,
                 ptr(cu_seqlens), ptr(start_pos), n_seqs, T, int(window or 0), float(scale), float(softcap or 0.0),
-                ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, ptr(out), n_heads, n_kv_heads, key_dim,
-                ptr(tc_status_word(q.device)), stream())
+                ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, ptr(part_acc if unmerged else out),
+                int(unmerged), n_heads, n_kv_heads, key_dim, ptr(tc_status_word(q.device)), stream())
             if st != NOT_SUPPORTED:
                 check(st, "flash_prefill_tc_ext")
         if st == NOT_SUPPORTED:
             st = core().tq_flash_prefill_ext(
                 ptr(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages), ptr(block_table), table_width,
                 ring_pages, page_tokens, ptr(cu_seqlens), ptr(start_pos), n_seqs, T, int(window or 0), float(scale),
-                float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, ptr(out), n_heads, n_kv_heads,
-                key_dim, stream())
+                float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld,
+                ptr(part_acc if unmerged else out), int(unmerged), n_heads, n_kv_heads, key_dim, stream())
             if st != NOT_SUPPORTED:
                 check(st, "flash_prefill_ext")
         if st != NOT_SUPPORTED:
+            if unmerged:
+                return part_acc, None, 1
             if gate is not None and not gate_ok:
                 from .elementwise import sigmoid_gate
                 sigmoid_gate(out, gate)
@@ -227,6 +238,8 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
             ptr(out), ptr(part_acc), ptr(part_ml), T, n_heads, n_kv_heads, key_dim, n_splits, stream())
         if st != NOT_SUPPORTED:
             check(st, "flash_decode_ext")
+            if unmerged:
+                return part_acc, part_ml, n_splits
             if n_splits > 1:
                 check(core().tq_attention_merge(ptr(part_acc), ptr(part_ml), ptr(out), dtype_code(out), T, n_heads,
                                                 value_dim, n_splits, ptr(sink), stream()), "attention_merge")
@@ -239,7 +252,9 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
         table_width, ring_pages, page_tokens, ptr(tok_pos), ptr(tok_seq), ptr(cu_seqlens), ptr(start_pos),
         int(window or 0), float(scale), ptr(out), ptr(part_acc), ptr(part_ml), T, n_heads, n_kv_heads, key_dim,
         value_dim, float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), n_splits, stream()),
-        "attention_ext", 2 if n_splits > 1 else 1)
+        "attention_ext", 2 if n_splits > 1 and not unmerged else 1)
+    if unmerged:
+        return part_acc, part_ml, n_splits
     if gate is not None:
         from .elementwise import sigmoid_gate
         sigmoid_gate(out, gate)

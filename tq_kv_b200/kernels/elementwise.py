@@ -24,9 +24,9 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, status: 
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
-            rows: Optional[torch.Tensor] = None):
-    """out[r] = x[rows[r] or r] / sqrt(mean(x^2) + eps) * weight.  x float32
-    [*, H]; weight float32 [H]; out float32 or bfloat16 [R, H]."""
+            rows: Optional[torch.Tensor] = None, centered: bool = False):
+    """out[r] = x[rows[r] or r] / sqrt(mean(x^2) + eps) * weight; with `centered` the row's mean is taken off first
+    (the layer norm).  x float32 [*, H]; weight float32 [H]; out float32 or bfloat16 [R, H]."""
     H = x.shape[-1]
     R = out.shape[0]
     if x.dtype != torch.float32 or weight.dtype != torch.float32 or weight.shape[0] != H or out.shape[-1] != H:
@@ -36,8 +36,9 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
     if rows is not None and (rows.dtype != torch.int32 or rows.shape[0] != R):
         raise KernelError("rmsnorm: rows must be int32 [R]")
     need_contiguous(x=x, weight=weight, out=out, rows=rows)
-    check(core().tq_rmsnorm(ptr(x), ptr(weight), ptr(out), dtype_code(out), ptr(rows), R, H, float(eps), stream()),
-          "rmsnorm")
+    kernel = core().tq_layernorm if centered else core().tq_rmsnorm
+    check(kernel(ptr(x), ptr(weight), ptr(out), dtype_code(out), ptr(rows), R, H, float(eps), stream()),
+          "layernorm" if centered else "rmsnorm")
     return out
 
 
@@ -235,7 +236,8 @@ def head_encode(proj: torch.Tensor, ctx_pos, q_out: torch.Tensor, *, q_col: int,
                 n_heads: int, n_kv_heads: int, key_dim: int, value_dim: int, cos=None, sin=None, rotary_dim: int = 0,
                 norm_eps: float = 0.0, k_out=None, v_out=None, k_pages=None, v_pages=None, block_table=None,
                 table_width: int = 0, ring_pages: int = 0, page_tokens: int = 64, paired: bool = False,
-                row_inv=None, q_weight=None, k_weight=None, v_scale: float = 1.0):
+                row_inv=None, q_weight=None, k_weight=None, v_scale: float = 1.0, maps: int = 1,
+                key_row: Optional[int] = None, value_row: Optional[int] = None):
     """From projected float32 rows [T, ld] (q heads from column q_col, k heads from k_col, v heads from v_col; with
     v_col < 0 the values are the keys as projected) to encoded q, and k / v packed and / or appended to the cache
     (see csrc/head_encode.cu).  `ctx_pos` = (tok_pos, tok_seq, new_lens).  q and k are rotated over their first
@@ -244,7 +246,11 @@ def head_encode(proj: torch.Tensor, ctx_pos, q_out: torch.Tensor, *, q_col: int,
     `row_inv` (float32 [T, 2] from `row_inv_rms`) and the weights q_weight [n_heads * key_dim] and k_weight
     [n_kv_heads * key_dim], q and k are first normed over their whole rows; with norm_eps and weights [key_dim] (shared
     by the heads) each head is normed and weighted before it is rotated.  The values leave times `v_scale`.
-    n_kv_heads may be 0: only q is encoded."""
+    n_kv_heads may be 0: only q is encoded.  `maps` > 1: every q and k head is that many vectors of key_dim, each
+    normed and rotated for itself; a key row holds a head's maps side by side, and every map's query becomes a head of
+    its own (head h's map m is head h * maps + m) whose row is zero but for its map's place, so that its product with a
+    key row is its map's score.  Rows are key_row and value_row wide (default maps * key_dim and value_dim), filled up
+    with zeros."""
     tok_pos, tok_seq, new_lens = ctx_pos
     T, ld = proj.shape
     if proj.dtype != torch.float32 or proj.stride(1) != 1:
@@ -255,7 +261,17 @@ def head_encode(proj: torch.Tensor, ctx_pos, q_out: torch.Tensor, *, q_col: int,
             raise KernelError(f"head_encode: rotary_dim {rotary_dim} needs float32 tables [positions, {rotary_dim // 2}]")
     if n_kv_heads and v_col < 0 and value_dim != key_dim:
         raise KernelError("head_encode: values that are the keys have the keys' width")
-    need = max(q_col + n_heads * key_dim, k_col + n_kv_heads * key_dim, v_col + n_kv_heads * value_dim if v_col >= 0 else 0)
+    key_row, value_row = key_row or maps * key_dim, value_row or value_dim
+    if maps < 1 or key_row < maps * key_dim or value_row < value_dim:
+        raise KernelError(f"head_encode: rows of {key_row} / {value_row} do not hold {maps} x {key_dim} / {value_dim}")
+    if (maps > 1 or key_row != key_dim or value_row != value_dim) and (v_col < 0 or row_inv is not None):
+        raise KernelError("head_encode: several maps or widened rows take values and norms of their own")
+    for name, t, width in (("q_out", q_out, n_heads * maps * key_row), ("k_out", k_out, n_kv_heads * key_row),
+                           ("v_out", v_out, n_kv_heads * value_row)):
+        if t is not None and (t.shape[0] != T or t.shape[1] != width):
+            raise KernelError(f"head_encode: {name} has shape {tuple(t.shape)}, expected [{T}, {width}]")
+    need = max(q_col + n_heads * maps * key_dim, k_col + n_kv_heads * maps * key_dim,
+               v_col + n_kv_heads * value_dim if v_col >= 0 else 0)
     if need > ld or min(q_col, k_col) < 0:
         raise KernelError(f"head_encode: the columns reach {need}, the rows have {ld}")
     for t in (k_out, v_out, k_pages, v_pages):
@@ -279,7 +295,8 @@ def head_encode(proj: torch.Tensor, ctx_pos, q_out: torch.Tensor, *, q_col: int,
                                 float(norm_eps), ptr(tok_pos), ptr(tok_seq), ptr(new_lens), ptr(block_table),
                                 table_width, ring_pages, page_tokens, ptr(q_out), ptr(k_out), ptr(v_out), ptr(k_pages),
                                 ptr(v_pages), dtype_code(q_out), T, n_heads, n_kv_heads, key_dim, value_dim,
-                                ptr(row_inv), ptr(q_weight), ptr(k_weight), int(bool(paired)), float(v_scale), stream()),
+                                ptr(row_inv), ptr(q_weight), ptr(k_weight), int(bool(paired)), float(v_scale), int(maps),
+                                key_row, value_row, stream()),
           "head_encode")
     return q_out
 
@@ -323,12 +340,38 @@ def round_rows(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def difference_of_maps(a: torch.Tensor, out: torch.Tensor, *, heads: int, row: int, value_dim: int, factor: float,
+                       eps: float, out_scale: float, gate: Optional[torch.Tensor] = None,
+                       ml: Optional[torch.Tensor] = None, n_splits: int = 1):
+    """out[t, h] = o / sqrt(mean(o^2) + eps) * out_scale (* sigmoid(gate[t, h])), o = a[t, 2h] - factor * a[t, 2h + 1]
+    over a head's value_dim entries.  `a` float32: the results of attention heads in rows of `row` entries, [T, 2 * heads *
+    row]; or with `ml` the unnormalised parts that the attention kernels leave per split of the keys (float32 [T, 2 *
+    heads, n_splits, row] and their maxima and sums [T, 2 * heads, n_splits, 2]), which are merged on the way.  gate
+    float32 [T, heads], possibly a column slice; out [T, heads * value_dim] float32 or bfloat16."""
+    T = out.shape[0]
+    if tuple(out.shape) != (T, heads * value_dim) or row < value_dim:
+        raise KernelError("difference_of_maps: out must be [T, heads * value_dim]")
+    if a.dtype != torch.float32 or a.numel() < T * 2 * heads * n_splits * row or (ml is None and n_splits != 1):
+        raise KernelError("difference_of_maps: a must hold float32 rows of both maps")
+    if ml is not None and (ml.dtype != torch.float32 or ml.numel() < T * 2 * heads * n_splits * 2):
+        raise KernelError("difference_of_maps: ml must hold a maximum and a sum per split")
+    if gate is not None and (gate.dtype != torch.float32 or tuple(gate.shape) != (T, heads) or gate.stride(1) != 1):
+        raise KernelError("difference_of_maps: gate must be float32 [T, heads]")
+    need_contiguous(a=a, out=out, ml=ml)
+    check(core().tq_difference_of_maps(ptr(a), ptr(ml), n_splits, row, value_dim, heads, float(factor), float(eps),
+                                       float(out_scale), ptr(gate), 0 if gate is None else gate.stride(0), ptr(out),
+                                       dtype_code(out), T, stream()), "difference_of_maps")
+    return out
+
+
 def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor):
-    """x[t, i] *= sigmoid(gate[t, i]) in place; gate float32, possibly a column slice of wider rows."""
+    """x[t, i] *= sigmoid(gate[t, i]) in place, or with fewer gates than entries (one per head) sigmoid(gate[t, i // (n /
+    gates)]); gate float32, possibly a column slice of wider rows."""
     T, n = x.shape
-    if gate.dtype != torch.float32 or tuple(gate.shape) != (T, n) or gate.stride(1) != 1 or not x.is_contiguous():
-        raise KernelError("sigmoid_gate: gate must be float32 of x's shape, x contiguous")
-    check(core().tq_sigmoid_gate(ptr(x), dtype_code(x), ptr(gate), gate.stride(0), T, n, stream()), "sigmoid_gate")
+    if gate.dtype != torch.float32 or gate.shape[0] != T or n % gate.shape[1] or gate.stride(1) != 1 or not x.is_contiguous():
+        raise KernelError("sigmoid_gate: gate must be float32 [T, n] or [T, heads], x contiguous")
+    check(core().tq_sigmoid_gate(ptr(x), dtype_code(x), ptr(gate), gate.stride(0), T, n, n // gate.shape[1], stream()),
+          "sigmoid_gate")
     return x
 
 

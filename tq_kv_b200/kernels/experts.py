@@ -20,17 +20,21 @@ def table_choice(tokens: torch.Tensor, table: torch.Tensor, n_experts: int) -> t
     return choice
 
 
-def router_choice(logits: torch.Tensor, top: int, scale: float, floor: float) -> tuple[torch.Tensor, torch.Tensor]:
-    """From a router's float32 logits [T, E]: the `top` experts with the largest sigmoid(logit) per token
-    (int32 [T, top], the lowest index first among equals) and their weights scale * s / (sum of the chosen s +
-    floor) (float32 [T, top])."""
+def router_choice(logits: torch.Tensor, top: int, scale: float = 1.0, floor: float = 0.0,
+                  softmax: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
+    """From a router's float32 logits [T, E] (may be a column slice): the `top` experts with the largest s =
+    sigmoid(logit) per token (int32 [T, top], the lowest index first among equals) and their weights scale * s / (sum of
+    the chosen s + floor) (float32 [T, top]).  With `softmax` s = exp(logit): the weights are then scale times the softmax
+    over the chosen logits (floor 0)."""
     T, E = logits.shape
     if logits.dtype != torch.float32 or logits.stride(1) != 1 or not 1 <= top <= E:
         raise KernelError("router_choice: float32 logits [T, E], 1 <= top <= E")
+    if softmax and floor:
+        raise KernelError("router_choice: a softmax over the chosen logits has no floor")
     choice = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    check(core().tq_router_choice(ptr(logits), logits.stride(0), E, top, float(scale), float(floor), ptr(choice),
-                                  ptr(weights), T, stream()), "router_choice")
+    check(core().tq_router_choice(ptr(logits), logits.stride(0), E, top, float(scale), float(floor), int(softmax),
+                                  ptr(choice), ptr(weights), T, stream()), "router_choice")
     return choice, weights
 
 
@@ -66,13 +70,25 @@ def _check_weights(weights, choice):
         raise KernelError("routed_experts: weights float32 of choice's shape")
 
 
+def _check_shared(shared, shared_gate, y, weights) -> int:
+    """The row stride of the shared result's gate (0 without one)."""
+    if shared is None:
+        return 0
+    if (shared.dtype != torch.float32 or shared.shape != y.shape or not shared.is_contiguous() or shared_gate is None
+            or shared_gate.dtype != torch.float32 or tuple(shared_gate.shape) != (y.shape[0], 1) or weights is None):
+        raise KernelError("routed_experts: a shared result is float32 [T, W] with a float32 gate [T, 1], beside weighted experts")
+    return shared_gate.stride(0)
+
+
 def routed_experts_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, choice: torch.Tensor,
                         y: torch.Tensor, accumulate: bool, weights: Optional[torch.Tensor] = None,
-                        gated: bool = True) -> torch.Tensor:
+                        gated: bool = True, shared: Optional[torch.Tensor] = None,
+                        shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y (=, +=) mean over a token's experts e (with `weights` float32 [T, top]: the sum weighted by them) of
     w_down[e] (silu(gate[e] x) * (up[e] x)), every (token, expert)
     pair a row-times-matrix product of its own.  With `gated` False an expert is w_down[e] max(up[e] x, 0)^2 and
-    w_gate_up is [E, F, W].  x [T, W]; w_gate_up [E, 2F, W]; w_down [E, W, F];
+    w_gate_up is [E, F, W].  `shared` (float32 [T, W]) is added times sigmoid(shared_gate) (float32 [T, 1], may be a column
+    slice).  x [T, W]; w_gate_up [E, 2F, W]; w_down [E, W, F];
     choice int32 [T, top]; y float32 [T, W]."""
     T, W = x.shape
     E, F2, W2 = w_gate_up.shape
@@ -85,11 +101,13 @@ def routed_experts_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.
         raise KernelError("routed_experts: x must be contiguous along its rows")
     need_contiguous(w_gate_up=w_gate_up, w_down=w_down, choice=choice, y=y)
     _check_weights(weights, choice)
+    ldg = _check_shared(shared, shared_gate, y, weights)
     top = choice.shape[1]
     act = torch.empty((T * top, F), dtype=x.dtype, device=x.device)
     check(core().tq_routed_experts_rows(ptr(x), dtype_code(x), x.stride(0), ptr(w_gate_up), ptr(w_down),
                                         dtype_code(w_down), ptr(choice), ptr(weights), top, T, W, F, ptr(act), ptr(y),
-                                        int(accumulate), int(gated), stream()), "routed_experts_rows", 2)
+                                        int(accumulate), int(gated), ptr(shared), ptr(shared_gate), ldg, stream()),
+          "routed_experts_rows", 2)
     return y
 
 
@@ -106,7 +124,8 @@ def routed_tiles_ok(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tens
 
 def routed_experts_tiles(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, choice: torch.Tensor,
                          y: torch.Tensor, accumulate: bool, weights: Optional[torch.Tensor] = None,
-                         gated: bool = True) -> torch.Tensor:
+                         gated: bool = True, shared: Optional[torch.Tensor] = None,
+                         shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The same result as `routed_experts_rows` for many rows: the (token, expert) pairs are sorted by expert
     into a buffer in which every expert owns whole tiles of 128 rows; two tensor-core products over the whole
     buffer follow, in which each tile multiplies with its own expert's matrices (the first gates, silu(g) * u,
@@ -120,6 +139,7 @@ def routed_experts_tiles(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch
         raise KernelError("routed_experts: choice int32 [T, top], y float32 [T, W]")
     need_contiguous(w_gate_up=w_gate_up, w_down=w_down, choice=choice, y=y)
     _check_weights(weights, choice)
+    ldg = _check_shared(shared, shared_gate, y, weights)
     top = choice.shape[1]
     n_pairs = T * top
     max_tiles = n_pairs // TILE_ROWS + E
@@ -138,6 +158,6 @@ def routed_experts_tiles(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch
                                  2 if gated else 4, E * F2, F if gated else 0, ptr(tile_up), status, stream()), "routed_gate_up")
     check(lib.tq_gemm_tc_grouped(ptr(act), ptr(w_down), ptr(out), dtype_code(out), rows, W, F, F, F, W,
                                  0, E * W, 0, ptr(tile_down), status, stream()), "routed_down")
-    check(lib.tq_routed_combine(ptr(out), ptr(pos), ptr(weights), top, T, W, ptr(y), int(accumulate), stream()),
-          "routed_combine")
+    check(lib.tq_routed_combine(ptr(out), ptr(pos), ptr(weights), top, T, W, ptr(y), int(accumulate), ptr(shared),
+                                ptr(shared_gate), ldg, stream()), "routed_combine")
     return y

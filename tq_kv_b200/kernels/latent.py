@@ -100,9 +100,10 @@ def latent_heads(q: torch.Tensor, kfv: torch.Tensor, rows: torch.Tensor, q_out: 
 
 
 def latent_expand(lat: torch.Tensor, up_v: Optional[torch.Tensor], out: torch.Tensor, *, heads: int, kv_rank: int,
-                  row_width: int, value_dim: int, gate: Optional[torch.Tensor] = None):
+                  row_width: int, value_dim: int, gate: Optional[torch.Tensor] = None, head_gate: bool = False):
     """out[t, h] = up_v[h] lat[t, h, :kv_rank], times sigmoid(gate[t, h]) entry by entry.  lat [T, heads *
-    row_width]; up_v [heads * value_dim, kv_rank]; gate float32 [T, heads * value_dim] (may be a column slice);
+    row_width]; up_v [heads * value_dim, kv_rank]; gate float32 [T, heads * value_dim], with `head_gate` [T, heads], one
+    number per head (may be a column slice);
     out [T, heads * value_dim].  Without up_v (then kv_rank >= value_dim) a head's first value_dim entries pass,
     gated."""
     T = lat.shape[0]
@@ -115,10 +116,11 @@ def latent_expand(lat: torch.Tensor, up_v: Optional[torch.Tensor], out: torch.Te
         raise KernelError("latent_expand: up_v must be [heads * value_dim, kv_rank] of out's dtype")
     ldg = 0
     if gate is not None:
-        if gate.dtype != torch.float32 or tuple(gate.shape) != (T, heads * value_dim) or gate.stride(1) != 1:
-            raise KernelError("latent_expand: gate must be float32 [T, heads * value_dim]")
+        want = (T, heads if head_gate else heads * value_dim)
+        if gate.dtype != torch.float32 or tuple(gate.shape) != want or gate.stride(1) != 1:
+            raise KernelError(f"latent_expand: gate must be float32 {list(want)}")
         ldg = gate.stride(0)
     need_contiguous(lat=lat, up_v=up_v, out=out)        # (need_contiguous passes None)
-    check(core().tq_latent_expand(ptr(lat), heads, kv_rank, row_width, value_dim, ptr(up_v), ptr(gate), ldg, ptr(out),
+    check(core().tq_latent_expand(ptr(lat), heads, kv_rank, row_width, value_dim, ptr(up_v), ptr(gate), ldg, int(head_gate), ptr(out),
                                   dtype_code(out), T, stream()), "latent_expand")
     return out

@@ -12,7 +12,7 @@ from .gated_delta import GatedDeltaMixer
 from .latent_attention import LatentAttention
 from .min_gru import MinGRUMixer
 from .mlstm import MatrixMemoryMixer
-from .norm import DynamicTanhNorm, GroupRMSNorm, RMSNorm
+from .norm import DynamicTanhNorm, GroupRMSNorm, LayerNorm, RMSNorm
 from .position import RotaryHalved, RotaryTables
 from .side_by_side import SideBySideMixer
 from .sigmoid_attention import SigmoidAttention
@@ -23,6 +23,7 @@ from .softmax_attention import SoftmaxAttention
 from .registry import make_block, make_part, part_kinds, register_block, register_part, unregister_part
 
 register_part("rms_norm", RMSNorm, replace=True)
+register_part("layer_norm", LayerNorm, replace=True)
 register_part("group_rms_norm", GroupRMSNorm, replace=True)
 register_part("delta_rule_mixer", DeltaRuleMixer, replace=True)
 register_part("decayed_state_mixer", DecayedStateMixer, replace=True)
@@ -53,7 +54,7 @@ register_block("residual_streams", StreamsBlock, replace=True)
 register_block("postnorm_residual", PostnormResidualBlock, replace=True)
 
 __all__ = ["ChannelDeltaMixer", "DynamicTanhNorm", "MinGRUMixer", "PlainFeedForward", "SublayerResult", "MatrixMemoryMixer", "PostnormResidualBlock", "ResidualStreams", "SoftmaxAttention", "StreamConnection", "StreamsBlock", "TableExperts", "GatedDeltaMixer", "LatentAttention", "ParallelResidualBlock", "RotaryTables", "StateSpaceMixer", "DecayedStateMixer", "DeltaRuleMixer", "GroupRMSNorm", "SideBySideMixer", "SigmoidAttention",
-           "FeedForward", "GQAttention", "LMHead", "Mixer", "Norm", "Part", "PositionEncoding",
+           "FeedForward", "GQAttention", "LMHead", "LayerNorm", "Mixer", "Norm", "Part", "PositionEncoding",
            "PrenormResidualBlock", "RMSNorm", "RotaryHalved", "Runtime", "StepBatch", "StepContext", "SwiGLU",
            "TokenEmbedding", "WeightSpec", "float32_vector", "make_block", "make_part", "part_kinds",
            "register_block", "register_part", "unregister_part"]

@@ -68,6 +68,17 @@ class GroupRMSNorm(RMSNorm):
         return kernels.group_rmsnorm(x, self.weight, self.eps, out, groups=self.groups, rows=rows)
 
 
+class LayerNorm(RMSNorm):
+    """The norm with the row's mean taken off: c / sqrt(mean(c^2) + eps) * weight, c = x - mean(x); no bias."""
+    pending = None                      # the products fold in the RMS norm only
+    stream_args = None                  # ... and so do the residual streams' kernels
+
+    def forward(self, x, out_dtype, rows=None):
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, self.width), dtype=out_dtype, device=x.device)
+        return kernels.rmsnorm(x, self.weight, self.eps, out, rows, centered=True)
+
+
 class DynamicTanhNorm(Norm):
     """A norm without statistics: tanh(alpha * x) * weight + bias, entry by entry in float32; alpha is one learned
     number (tensor `<weight_name>.alpha`), weight and bias (`<weight_name>.b`) have the row's width."""

@@ -71,7 +71,7 @@ class RotaryTables(PositionEncoding):
     i + rotary_dim / 2).  The angles are formed in float64 on the host and their cosines and sines rounded once
     to float32, so that the tables carry no error that grows with the position.
 
-    Plain rates are theta^(-2i / rotary_dim).  With `scaling` = {factor F, original L, fast, slow} the slow
+    Plain rates are theta^(-2i / rotary_dim), divided by `rate_divisor` (1 by default) if that is given.  With `scaling` = {factor F, original L, fast, slow} the slow
     pairs are stretched for contexts longer than the L positions the rates were made for: a pair that makes t
     turns over L positions has index n(t) = rotary_dim * ln(L / (2 pi t)) / (2 ln theta); with
     lo = max(floor(n(fast)), 0) and hi = min(ceil(n(slow)), rotary_dim - 1), pair i takes the share
@@ -88,6 +88,9 @@ class RotaryTables(PositionEncoding):
             raise ValueError(f"rotary tables: layout '{self.layout}' (pairs or halves), an even rotary_dim")
         sc = self.params.get("scaling")
         self.scaling = None
+        self.rate_divisor = float(self.params.get("rate_divisor", 1.0))
+        if not self.rate_divisor > 0.0 or (sc and self.rate_divisor != 1.0):
+            raise ValueError(f"rotary tables: rate_divisor {self.rate_divisor} must be positive and stands alone")
         if sc:
             self.scaling = (float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"]))
             if min(self.scaling) <= 0.0:
@@ -105,7 +108,7 @@ class RotaryTables(PositionEncoding):
         i = torch.arange(half, dtype=torch.float64)
         rate = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / max(2, self.rotary_dim))
         if self.scaling is None:
-            return rate, 1.0
+            return rate / self.rate_divisor, 1.0
         import math
         F, L, fast, slow = self.scaling
 
@@ -118,7 +121,7 @@ class RotaryTables(PositionEncoding):
         return rate / F * share + rate * (1.0 - share), 0.1 * math.log(F) + 1.0
 
     def prepare(self, runtime: Runtime, shared: Optional[dict] = None) -> None:
-        key = (("rotary_tables", self.rotary_dim, self.theta, self.scaling), runtime.max_context, str(runtime.device))
+        key = (("rotary_tables", self.rotary_dim, self.theta, self.scaling, self.rate_divisor), runtime.max_context, str(runtime.device))
         if shared is not None and key in shared:
             self.cos, self.sin = shared[key]
             return

@@ -32,6 +32,12 @@
                     their true positions)
   output_gate       the heads side by side are multiplied entry by entry with
                     sigmoid(W_g x) before the output projection
+  head_gate         head h's result is multiplied by sigmoid((W_g x)_h), one number per head
+  difference        {"offset": d, "eps": e}: two attention maps per head over the same values.  q and
+                    k have twice the rows, head by head [map 1, map 2], each normed and rotated for
+                    itself; with a1 and a2 the maps' results and the layer's number
+                    lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + d  (tensors `lq1` .. `lk2` of the key
+                    width), o = a1 - lambda * a2, then o / sqrt(mean(o^2) + e) * (1 - d) per head
   result_scale      the mixer's result is multiplied by it: the values are, before they are
                     rounded and cached (the result is linear in them)
 Query head h reads key/value head h // (heads / kv_heads).  Key rows and value rows
@@ -46,6 +52,12 @@ first tokens are kept (the kernels skip what lies between the kept tokens and th
 window).  Scores, softmax and the bias are float32.  bfloat16 steps whose keys and
 values have one width run the tensor-core kernels (`kernels.attention_ext`), which
 also apply the output gate where they can.
+
+Two maps per head run through the same kernels as twice as many query heads: a key row holds both maps' keys side
+by side, a map's query is zero outside its map's place, so every key and value row is read once for both maps of
+all query heads that share it; the float32 results (in decoding the shares of the split key range) are merged,
+subtracted, normed, gated and rounded once by one kernel (`kernels.difference_of_maps`).  Rows are widened with
+zeros to a width of the tensor-core kernels where one holds both.
 """
 from __future__ import annotations
 
@@ -56,7 +68,7 @@ import torch
 from .. import kernels
 from ..cache import PAGE_TOKENS, KVRequest, ring_pages_for
 from ..config import ConfigError
-from .base import Mixer, Runtime, StepContext, WeightSpec, float32_vector
+from .base import Mixer, Runtime, StepContext, WeightSpec, float32_vector, stack_rows
 from .registry import make_part
 
 
@@ -85,6 +97,20 @@ class SoftmaxAttention(Mixer):
             raise ConfigError("softmax attention: heads need at least one entry")
         self.key_dim = -(-self.key_dim_given // 8) * 8
         self.value_dim = -(-self.value_dim_given // 8) * 8
+        self.difference = dict(p["difference"]) if p.get("difference") else None
+        self.maps = 2 if self.difference else 1
+        if self.difference:
+            # the encoding kernel pads the rows, not the weights
+            self.key_dim, self.value_dim = self.key_dim_given, self.value_dim_given
+            clash = [n for n in ("output_gate", "sink", "shared_kv", "row_norm_eps", "slope_exponent") if p.get(n)]
+            if clash or self.values != "projected" or float(p.get("result_scale", 1.0)) != 1.0:
+                raise ConfigError(f"softmax attention: a difference of two maps has values of its own and no "
+                                  f"{', '.join(clash) or 'result_scale'}")
+        rows = (-(-self.maps * self.key_dim // 8) * 8, -(-self.value_dim // 8) * 8)
+        if self.difference:                                  # one width of the tensor-core kernels for both, if there is one
+            width = next((w for w in kernels.TENSOR_CORE_WIDTHS if w >= max(rows)), None)
+            rows = rows if width is None else (width, width)
+        self.key_row, self.value_row = rows                  # widths of the rows the attention kernels see
         self.scale = float(p["scale"])
         self.softcap = float(p["softcap"]) if p.get("softcap") else None
         self.slope_exponent = float(p["slope_exponent"]) if p.get("slope_exponent") else None
@@ -124,7 +150,10 @@ class SoftmaxAttention(Mixer):
         self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
         self.output_gate = bool(p.get("output_gate", False))
         self.names = dict(p.get("names", {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o"}))
-        kernels.check_row_widths(self.n_heads, self.n_kv_heads, self.key_dim, self.value_dim)
+        kernels.check_row_widths(self.n_heads * self.maps, self.n_kv_heads, self.key_row, self.value_row)
+        self.head_gate = bool(p.get("head_gate", False))
+        if self.head_gate and self.output_gate:
+            raise ConfigError("softmax attention: a gate per entry or per head, not both")
         self.position = make_part(p["position"]) if p.get("position") is not None else None
         if self.position is not None:
             if getattr(self.position, "layout", None) not in ("halves", "pairs"):
@@ -134,8 +163,8 @@ class SoftmaxAttention(Mixer):
                                   f"{self.key_dim_given}")
         if self.qk_norm_eps and self.row_norm_eps:
             raise ConfigError("softmax attention: q and k are normed per head or over the whole row, not both")
-        self.q_width = self.n_heads * self.key_dim
-        self.k_width = 0 if self.shared_kv else self.n_kv_heads * self.key_dim
+        self.q_width = self.n_heads * self.maps * self.key_dim
+        self.k_width = 0 if self.shared_kv else self.n_kv_heads * self.maps * self.key_dim
         self.v_width = self.n_kv_heads * self.value_dim if self.values == "projected" and not self.shared_kv else 0
         self.o_width = self.n_heads * self.value_dim
         self.w_in = self.w_o = self.slopes = self.sinks = None
@@ -147,9 +176,9 @@ class SoftmaxAttention(Mixer):
 
     def weight_specs(self):
         d, e, H, G = self.key_dim_given, self.value_dim_given, self.n_heads, self.n_kv_heads
-        specs = [WeightSpec(self._n("q"), (H * d, self.hidden), "matrix")]
+        specs = [WeightSpec(self._n("q"), (H * self.maps * d, self.hidden), "matrix")]
         if not self.shared_kv:
-            specs.append(WeightSpec(self._n("k"), (G * d, self.hidden), "matrix"))
+            specs.append(WeightSpec(self._n("k"), (G * self.maps * d, self.hidden), "matrix"))
             if self.values == "projected":
                 specs.append(WeightSpec(self._n("v"), (G * e, self.hidden), "matrix"))
         if self.row_norm_eps:
@@ -160,8 +189,10 @@ class SoftmaxAttention(Mixer):
             specs += [WeightSpec(self._n("q_norm"), (d,), "norm_scale"), WeightSpec(self._n("k_norm"), (d,), "norm_scale")]
         if self.sink == "learned":
             specs.append(WeightSpec(self._n("sink"), (H,), "sink"))
-        if self.output_gate:
-            specs.append(WeightSpec(self._n("gate"), (H * e, self.hidden), "matrix"))
+        if self.difference:
+            specs += [WeightSpec(self._n(n), (d,), "map_weight") for n in ("lq1", "lk1", "lq2", "lk2")]
+        if self.output_gate or self.head_gate:
+            specs.append(WeightSpec(self._n("gate"), (H if self.head_gate else H * e, self.hidden), "matrix"))
         specs.append(WeightSpec(self._n("out"), (self.hidden, H * e), "matrix"))
         return specs
 
@@ -176,15 +207,16 @@ class SoftmaxAttention(Mixer):
 
     def bind(self, tensors, runtime: Runtime, shared: Optional[dict] = None):
         which = ["q"] + ([] if self.shared_kv else ["k"] + (["v"] if self.values == "projected" else [])) \
-            + (["gate"] if self.output_gate else [])
-        heads = {"q": (self.n_heads, self.key_dim_given, self.key_dim),
-                 "k": (self.n_kv_heads, self.key_dim_given, self.key_dim),
+            + (["gate"] if self.output_gate or self.head_gate else [])
+        heads = {"q": (self.n_heads * self.maps, self.key_dim_given, self.key_dim),
+                 "k": (self.n_kv_heads * self.maps, self.key_dim_given, self.key_dim),
                  "v": (self.n_kv_heads, self.value_dim_given, self.value_dim),
-                 "gate": (self.n_heads, self.value_dim_given, self.value_dim)}
-        ws = [self._pad_heads(tensors[self._n(x)], *heads[x]) for x in which]
-        if len({w.dtype for w in ws}) != 1:
-            ws = [w.to(torch.float32) for w in ws]
-        self.w_in = torch.cat(ws, dim=0).contiguous()        # one product: [q | k | (v) | (gate)]
+                 "gate": (self.n_heads,) + ((1, 1) if self.head_gate else (self.value_dim_given, self.value_dim))}
+        self.w_in, _ = stack_rows([self._pad_heads(tensors[self._n(x)], *heads[x]) for x in which])
+        # one product: [q | k | (v) | (gate)]
+        if self.difference:
+            lq1, lk1, lq2, lk2 = (tensors[self._n(n)].detach().to("cpu", torch.float64) for n in ("lq1", "lk1", "lq2", "lk2"))
+            self.factor = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + float(self.difference["offset"])
         w_o = tensors[self._n("out")]
         if self.value_dim != self.value_dim_given:           # zero columns where the heads were padded
             w_o = self._pad_heads(w_o.t(), self.n_heads, self.value_dim_given, self.value_dim).t()
@@ -229,8 +261,8 @@ class SoftmaxAttention(Mixer):
     def cache_request(self):
         if self.shared_kv:
             return None
-        return KVRequest(self.n_kv_heads, self.key_dim, self.cache_window if self._ring else None,
-                         self.value_dim if self.value_dim != self.key_dim else None)
+        return KVRequest(self.n_kv_heads, self.key_row, self.cache_window if self._ring else None,
+                         self.value_row if self.value_row != self.key_row else None)
 
     def _use_packed(self, start_pos, step_lens, owns_cache) -> bool:
         """Prompts that start at position 0 attend over the step's own keys: their own, or (a layer that reads
@@ -266,13 +298,13 @@ class SoftmaxAttention(Mixer):
         act = ctx.runtime.act_dtype
         owns = kv is not None and kv.writes and not self.shared_kv
         packed = self._use_packed(b.host_start, b.host_lens, owns)
-        q = torch.empty((T, self.q_width), dtype=act, device=dev)
+        q = torch.empty((T, self.n_heads * self.maps * self.key_row), dtype=act, device=dev)
         k = v = None
         if packed and self.shared_kv:
             k, v = ctx.step_shared[("packed_kv", ctx.cache_entry)]
         elif packed:
-            k = torch.empty((T, self.k_width), dtype=act, device=dev)
-            v = torch.empty((T, self.n_kv_heads * self.value_dim), dtype=act, device=dev)
+            k = torch.empty((T, self.n_kv_heads * self.key_row), dtype=act, device=dev)
+            v = torch.empty((T, self.n_kv_heads * self.value_row), dtype=act, device=dev)
             if self.shares_packed and ctx.step_shared is not None:
                 ctx.step_shared[("packed_kv", ctx.entry)] = (k, v)
         pos = self.position
@@ -285,7 +317,8 @@ class SoftmaxAttention(Mixer):
             proj, (b.tok_pos, b.tok_seq, b.new_lens), q, q_col=0, k_col=self.k_col, v_col=self.v_col,
             n_heads=self.n_heads, n_kv_heads=0 if self.shared_kv else self.n_kv_heads, key_dim=self.key_dim,
             value_dim=self.value_dim, row_inv=row_inv, q_weight=self.q_norm_w, k_weight=self.k_norm_w,
-            paired=pos is not None and pos.paired, v_scale=self.result_scale,
+            paired=pos is not None and pos.paired, v_scale=self.result_scale, maps=self.maps, key_row=self.key_row,
+            value_row=self.value_row,
             cos=pos.cos if pos is not None else None, sin=pos.sin if pos is not None else None,
             rotary_dim=pos.rotary_dim if pos is not None else 0, norm_eps=self.qk_norm_eps,
             k_out=None if self.shared_kv else k, v_out=None if self.shared_kv else v,
@@ -294,24 +327,35 @@ class SoftmaxAttention(Mixer):
             ring_pages=kv.ring_pages if owns else 0, page_tokens=kv.page_tokens if kv is not None else PAGE_TOKENS)
         kernels.mark("rotary")
         out = torch.empty((T, self.o_width), dtype=act, device=dev)
-        common = dict(n_heads=self.n_heads, n_kv_heads=self.n_kv_heads, key_dim=self.key_dim,
-                      value_dim=self.value_dim, tok_pos=b.tok_pos, tok_seq=b.tok_seq, cu_seqlens=b.cu_seqlens,
+        gate = proj[:, self.g_col:self.g_col + (self.n_heads if self.head_gate else self.o_width)] \
+            if self.output_gate or self.head_gate else None
+        common = dict(n_heads=self.n_heads * self.maps, n_kv_heads=self.n_kv_heads, key_dim=self.key_row,
+                      value_dim=self.value_row, tok_pos=b.tok_pos, tok_seq=b.tok_seq, cu_seqlens=b.cu_seqlens,
                       start_pos=b.start_pos, scale=self.scale, window=self.window, keep_first=self.keep_first,
                       softcap=self.softcap, slopes=self.slopes, chunk=self.chunk,
                       sink=self.sinks if self.sinks is not None else False,
-                      gate=proj[:, self.g_col:self.g_col + self.o_width] if self.output_gate else None)
+                      gate=gate if self.output_gate else None, unmerged=self.difference is not None)
+        into = None if self.difference else out
         if packed:
-            kernels.attention_ext(q, out, k_packed=k, v_packed=v, **common)
+            parts = kernels.attention_ext(q, into, k_packed=k, v_packed=v, **common)
         else:
             max_keys = b.max_new_len if self.span is None else min(b.max_new_len, self.span + self.keep_first)
             n_splits = kernels.plan_splits(T, self.n_kv_heads, max_keys, ctx.runtime.sm_count)
             scratch = None
             if n_splits > 1:
-                scratch = torch.empty(kernels.split_scratch_floats(T, self.n_heads, self.value_dim, n_splits),
+                scratch = torch.empty(kernels.split_scratch_floats(T, self.n_heads * self.maps, self.value_row, n_splits),
                                       dtype=torch.float32, device=dev)
-            kernels.attention_ext(q, out, k_pages=kv.k_pages, v_pages=kv.v_pages, block_table=kv.block_table,
-                                  table_width=kv.table_width, ring_pages=kv.ring_pages, page_tokens=kv.page_tokens,
-                                  n_splits=n_splits, scratch=scratch, **common)
+            parts = kernels.attention_ext(q, into, k_pages=kv.k_pages, v_pages=kv.v_pages, block_table=kv.block_table,
+                                          table_width=kv.table_width, ring_pages=kv.ring_pages, page_tokens=kv.page_tokens,
+                                          n_splits=n_splits, scratch=scratch, **common)
         kernels.mark("attention")
+        if self.difference:
+            sums, ml, n = parts
+            kernels.difference_of_maps(sums, out, heads=self.n_heads, row=self.value_row, value_dim=self.value_dim,
+                                       factor=self.factor, eps=float(self.difference["eps"]),
+                                       out_scale=1.0 - float(self.difference["offset"]), gate=gate, ml=ml, n_splits=n)
+            kernels.mark("difference")
+        elif self.head_gate:
+            kernels.sigmoid_gate(out, gate)
         kernels.linear(out, self.w_o, out=residual, accumulate=accumulate)
         kernels.mark("o")

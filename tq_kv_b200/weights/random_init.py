@@ -2,7 +2,7 @@
 a model folder (config.json + model.safetensors) that the loader reads back.
 
 Init rules by role: matrices and embeddings N(0, 0.02^2); biases N(0, 0.02^2);
-norm scales 1 + N(0, 0.1^2) (N(0, 0.1^2) where the model adds the one itself); the taps of short convolutions N(0, 0.3^2); the alpha of a Dynamic Tanh norm 0.5 + N(0, 0.05^2); sinks N(0, 0.5^2).  The generator is counter-based: element i of a
+norm scales 1 + N(0, 0.1^2) (N(0, 0.1^2) where the model adds the one itself); the taps of short convolutions N(0, 0.3^2); the alpha of a Dynamic Tanh norm 0.5 + N(0, 0.05^2); sinks N(0, 0.5^2); the vectors that weigh the second of two attention maps N(0, 0.1^2).  The generator is counter-based: element i of a
 tensor depends on (seed, tensor name, i) only, so a tensor's values depend
 neither on which other tensors exist nor on where they are made.  The host
 twin below (numpy) and the device kernel (csrc/random_fill.cu) do the same
@@ -24,7 +24,7 @@ import torch
 from .safetensors_io import write_safetensors
 
 _STD = {"matrix": 0.02, "embedding": 0.02, "bias": 0.02, "norm_scale": 0.1, "norm_offset": 0.1, "conv": 0.3,
-        "stream_read": 0.1, "stream_write": 0.1, "stream_mix": 0.1, "tanh_alpha": 0.05, "sink": 0.5}
+        "stream_read": 0.1, "stream_write": 0.1, "stream_mix": 0.1, "tanh_alpha": 0.05, "sink": 0.5, "map_weight": 0.1}
 _OFFSET = {"norm_scale": 1.0, "stream_write": 1.0, "tanh_alpha": 0.5}
 _HOST_MADE = ("stream_read", "stream_write", "stream_mix", "tanh_alpha")      # a few numbers: made on the host for every device
 CHOICE_TABLE = "choice_table:"      # role "choice_table:<E>": int32 rows of distinct indices below E
