@@ -26,13 +26,13 @@ then 256 decode steps.  Peaks come from MEASURED_PEAKS.json beside this file
 if it exists, else from an earlier measurement on the same kind of machine
 (6.65 TB/s, 1.59 PFLOP/s).
 
-`--design zodosun|rirudra|pavisun|furesun|gokapel [--sizes 1k,2k,4k] [--prompt 2048]` is another program: the named decoder beside the Qwen2
+`--design zodosun|rirudra|pavisun|furesun|gokapel|safurax [--sizes 1k,2k,4k] [--prompt 2048]` is another program: the named decoder beside the Qwen2
 decoder of the same width, depth, heads, feed-forward and vocabulary (random weights, bfloat16): device time of a
 prompt, of decode steps at batch 8 and 64, and the time by class of kernel with what the attention and scan
 kernels reach of their rooflines, as one JSON line of its own (`--design rirudra` also runs the Zodosun decoder,
 whose scans are the like kernels of its own; `--design pavisun` runs the Pavisun decoder and the Qwen2 decoder only;
 `--design furesun` runs the Furesun, Rirudra and Qwen2 decoders; `--design gokapel` the Gokapel, Rirudra, Pavisun and
-Qwen2 decoders).  The default workload and its line are untouched.
+Qwen2 decoders; `--design safurax` the Safurax, Furesun and Qwen2 decoders).  The default workload and its line are untouched.
 
 The reference arm (`--impl reference`) cannot run here: the reference is a
 Rust workspace and no Rust toolchain is installed, so it prints its
@@ -377,6 +377,105 @@ def gokapel_roofline(rec: dict, pk: dict, P: int, sms: int) -> dict:
     return roof
 
 
+SAFURAX_WINDOW, SAFURAX_EXPERTS, SAFURAX_TOP = 1024, 8, 2
+
+
+def safurax_config(width: int, ff: int, layers: int, vocab: int) -> dict:
+    """A Safurax configuration of the given width: a difference of two maps of 64 over values of 128 on a quarter as many
+    key/value heads, with a dense feed-forward; attention through a latent of 128 values without positions, queries
+    through a latent of half the width; attention through a latent of 96 values and a rotated part of 32 (a window of
+    1,024, a sink, a gate per head); the same reading the third layer's latents; the last three layers with 8 experts
+    of a quarter of the feed-forward width of which a token uses 2, and a gated shared expert of half of it (as many
+    products per token as the dense feed-forward has)."""
+    heads, kv = width // 128, max(1, width // 512)
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 2},
+           "router": {"experts": SAFURAX_EXPERTS, "top": SAFURAX_TOP}}
+    maps = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5,
+            "rot": {"base": 1e4, "dims": 64, "scaling": {"factor": 4.0}}}
+    plain = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 128, "q_rank": width // 2, "scale": 128 ** -0.5}
+    windowed = {"heads": heads, "dim": 96, "rot_dim": 32, "vdim": 128, "kv_rank": 96, "scale": 128 ** -0.5,
+                "mask": {"size": SAFURAX_WINDOW}, "rot": {"base": 1e4, "dims": 32}}
+    order = [("attention", maps, {"kind": "dense", "ff": ff}), ("latent_attention", plain, moe),
+             ("latent_attention_2", windowed, moe), ("latent_attention_2", {**windowed, "kv_from": 2}, moe)]
+    return {"architecture": "Safurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 3.0},
+            "max_positions": 8192, "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in order[:layers]]}
+
+
+def safurax_roofline(rec: dict, pk: dict, P: int, sms: int) -> dict:
+    """What the classes of the Safurax decoder reach of their rooflines, beside the like classes of the Furesun decoder
+    (latent attention, experts) and of the Qwen2 decoder (attention, products, norms)."""
+    width, ff, layers = rec["width"], rec["ff"], rec["layers"]
+    heads, kv, d = width // 128, max(1, width // 512), 128
+    s, f, q = rec["safurax"], rec["furesun"], rec["qwen2"]
+    roof: dict = {}
+
+    def us(model, when, names):
+        return sum(model[when].get(k, 0.0) for k in names) * 1e-6
+
+    def tensor(name, flops, model, when, names):
+        roof[name + ".frac_of_bf16"] = round(flops / us(model, when, names) / 1e12 / pk["bf16_tflops"], 3)
+
+    def hbm(name, nbytes, model, when, names):
+        roof[name + ".frac_of_hbm"] = round(nbytes / us(model, when, names) / 1e9 / pk["hbm_gbs"], 3)
+
+    pre, dec = "prefill_classes_us", "decode_b64_classes_us"
+    pairs, Wd, E = P * (P + 1) / 2, SAFURAX_WINDOW, SAFURAX_EXPERTS
+    seen = sum(min(i + 1, Wd) for i in range(P))
+    # the maps' scores (two of 64 entries) and their sums of values (two of 128), the plain latent and two windowed ones
+    tensor("safurax.prefill.attention", heads * ((4 * 64 + 4 * d) * pairs + 4 * d * (pairs + 2 * seen)), s, pre, ["attention"])
+    tensor("furesun.prefill.attention", 4 * heads * d * seen * 3, f, pre, ["attention"])
+    tensor("qwen2.prefill.attention", 4 * heads * d * pairs * layers, q, pre, ["attention"])
+    # two float32 results per head in, one rounded row out
+    hbm("safurax.prefill.difference", P * heads * d * (2 * 4 + 2), s, pre, ["difference"])
+    # encodings.  Maps: the float32 projections read, two widened queries per head, keys and values (rows and pages)
+    # written.  Latents: float32 projections read, rounded ones written; the windowed layers' heads (q, k, v float32 in,
+    # bfloat16 out) and their gated, narrowed results
+    maps = (heads + 2 * kv) * d * 4 + 2 * heads * d * 2 + 2 * 2 * kv * d * 2
+    lat1 = (width // 2 + 128) * (4 + 2) + 128 * 2
+    lat2 = heads * (128 + 96 + 128) * 4 + 3 * heads * d * 2
+    hbm("safurax.prefill.encodings", P * (maps + lat1 + 2 * lat2 + 128 * (4 + 2 + 2)), s, pre, ["rotary"])
+    f_attn = (heads + 2 * kv) * d * 4 + (heads + 4 * kv) * d * 2 + heads * d * (4 + 2)
+    hbm("furesun.prefill.encodings", P * (f_attn + lat2 + 128 * (4 + 2 + 2) + heads * d * 4), f, pre, ["rotary"])
+    n_in = [(heads + 2 * kv) * d + heads, width // 2 + 128, heads * d + 128 + heads, heads * d + heads]
+    up1, up2 = width // 2 * heads * d + 2 * 128 * heads * d, 96 * heads * (96 + 128)
+    tensor("safurax.prefill.qkv", 2 * P * (width * sum(n_in) + up1 + 2 * up2), s, pre, ["qkv"])
+    tensor("qwen2.prefill.qkv", 2 * P * width * (heads + 2 * kv) * d * layers, q, pre, ["qkv"])
+    tensor("safurax.prefill.o", 2 * P * width * heads * d * 4, s, pre, ["o"])
+    tensor("qwen2.prefill.o", 2 * P * width * heads * d * layers, q, pre, ["o"])
+    ff_flops = 6 * P * width * ff
+    tensor("safurax.prefill.dense_feed_forward", ff_flops, s, pre, ["gate_up", "down"])
+    tensor("furesun.prefill.dense_feed_forward", ff_flops, f, pre, ["gate_up", "down"])
+    tensor("qwen2.prefill.dense_feed_forward", ff_flops * layers, q, pre, ["gate_up", "down"])
+    tensor("safurax.prefill.experts", ff_flops * 3 / 2, s, pre, ["experts", "router"])
+    tensor("furesun.prefill.experts", ff_flops * 3 / 2, f, pre, ["experts"])
+    tensor("safurax.prefill.shared_expert", ff_flops * 3 / 2, s, pre, ["shared_expert"])
+    tensor("furesun.prefill.shared_expert", ff_flops * 3 / 2, f, pre, ["shared_expert"])
+    hbm("safurax.prefill.norms", P * width * (4 + 2) * 2 * 4, s, pre, ["norms"])
+    hbm("qwen2.prefill.norms", P * width * (4 + 2) * 2 * layers, q, pre, ["norms"])
+    n = P + 16
+    row = 2 * kv * d * 2
+    hbm("safurax.decode_b64.attention", 64 * (n * row + n * 128 * 2 + 2 * min(n, Wd) * 128 * 2), s, dec, ["attention"])
+    hbm("furesun.decode_b64.attention", 64 * min(n, Wd) * (128 * 2 + 2 * row), f, dec, ["attention"])
+    hbm("qwen2.decode_b64.attention", 64 * n * row * layers, q, dec, ["attention"])
+    # decode: the latents' per-head matrices read once (they ride in this class), float32 projections and rounded rows
+    up = 2 * heads * d * (2 * 128 + 2 * 2 * 96)
+    act = 64 * heads * 3 * (4 * 128 + 2 * 128 * 3)
+    hbm("safurax.decode_b64.encodings", up + act + 64 * maps, s, dec, ["rotary"])
+    hbm("furesun.decode_b64.encodings", 2 * heads * d * 2 * 96 + act // 3 + 64 * f_attn, f, dec, ["rotary"])
+    hbm("safurax.decode_b64.products", 2 * (width * (sum(n_in) + 4 * heads * d) + width // 2 * heads * d), s, dec, ["qkv", "o"])
+    hbm("qwen2.decode_b64.products", 2 * width * ((heads + 2 * kv) * d + heads * d) * layers, q, dec, ["qkv", "o"])
+    hbm("safurax.decode_b64.dense_feed_forward", 3 * width * ff * 2, s, dec, ["gate_up", "down"])
+    hbm("furesun.decode_b64.dense_feed_forward", 3 * width * ff * 2, f, dec, ["gate_up", "down"])
+    hbm("qwen2.decode_b64.dense_feed_forward", 3 * width * ff * 2 * layers, q, dec, ["gate_up", "down"])
+    hbm("safurax.decode_b64.experts", 3 * width * (ff // 4) * E * 2 * 3, s, dec, ["experts", "router"])
+    hbm("furesun.decode_b64.experts", 3 * width * (ff // 4) * E * 2 * 3, f, dec, ["experts"])
+    hbm("safurax.decode_b64.shared_expert", 3 * width * (ff // 2) * 2 * 3, s, dec, ["shared_expert"])
+    hbm("furesun.decode_b64.shared_expert", 3 * width * (ff // 2) * 2 * 3, f, dec, ["shared_expert"])
+    hbm("safurax.decode_b64.norms", 64 * width * (4 + 2) * 2 * 4, s, dec, ["norms"])
+    hbm("qwen2.decode_b64.norms", 64 * width * (4 + 2) * 2 * layers, q, dec, ["norms"])
+    return roof
+
+
 def furesun_roofline(rec: dict, pk: dict, P: int, sms: int) -> dict:
     """What the classes of the Furesun decoder reach of their rooflines, beside the like classes of the Qwen2
     decoder (attention, feed-forward, the kernels between the sublayers) and of the Rirudra decoder (the scan)."""
@@ -549,6 +648,9 @@ def design_compare(args) -> int:
                 models = [("gokapel", gokapel_config(width, ff, layers, vocab)),
                           ("rirudra", rirudra_config(width, ff, layers, vocab)),
                           ("pavisun", pavisun_config(width, ff, layers, vocab)), ("qwen2", qwen)]
+            if args.design == "safurax":
+                models = [("safurax", safurax_config(width, ff, layers, vocab)),
+                          ("furesun", furesun_config(width, ff, layers, vocab)), ("qwen2", qwen)]
             for model, cfg in models:
                 eng = tq.Engine.from_random(cfg, seed=0, dtype="bfloat16", max_slots=64, max_context=ctx,
                                             max_tokens=64 * ctx)
@@ -625,6 +727,9 @@ def design_compare(args) -> int:
             if args.design == "gokapel":
                 rec["roofline"] = gokapel_roofline(rec, pk, P, sms)
                 continue
+            if args.design == "safurax":
+                rec["roofline"] = safurax_roofline(rec, pk, P, sms)
+                continue
             # what the classes reach of their rooflines
             heads, d = width // 128, 128
             z, q = rec["zodosun"], rec["qwen2"]
@@ -657,7 +762,7 @@ def design_compare(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["zodosun", "rirudra", "pavisun", "furesun", "gokapel"],
+    ap.add_argument("--design", default=None, choices=["zodosun", "rirudra", "pavisun", "furesun", "gokapel", "safurax"],
                     help="instead of the default workload: this design beside the Qwen2 decoder of equal size")
     ap.add_argument("--sizes", default="1k,2k,4k", help="with --design: which of the sizes 1k, 2k, 4k (the model's width)")
     ap.add_argument("--gpus", type=int, default=1)
