@@ -234,6 +234,102 @@ def test_a_learned_sink_over_a_cache_whose_values_are_its_keys(H, row, dtype, wi
                 _close(out.reshape(H, row), want[t], tol, f"row {t}, fast={fast}, {n_splits} splits")
 
 
+# ---- many prompts at once -------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("sink", [False, True])
+def test_prompt_attention_under_load(sink):
+    """Many more tiles than fit the device, over and over, with the values cold and the keys warm in the cache: a block
+    whose first value tile comes late has scores of two tiles ready before its first product with values, and must
+    neither wait for good nor mix tiles up."""
+    from tq_kv_b200 import kernels
+    H, d, n_seqs, L = 8, 128, 8, 1024
+    T = n_seqs * L
+    g = torch.Generator(device=DEV).manual_seed(1)
+    q, k, v = (torch.randn(T, H * d, generator=g, device=DEV).to(torch.bfloat16) for _ in range(3))
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=DEV)
+    pos = _ints(list(range(L)) * n_seqs)
+    seq = _ints([b for b in range(n_seqs) for _ in range(L)])
+    args = dict(n_heads=H, n_kv_heads=H, tok_pos=pos, tok_seq=seq, cu_seqlens=_ints([b * L for b in range(n_seqs + 1)]),
+                start_pos=_ints([0] * n_seqs), window=None, scale=d ** -0.5, k_packed=k, v_packed=v)
+    sinks = torch.full((H,), 1.0, device=DEV)
+    first = None
+    for i in range(250):
+        if i % 5 == 0:
+            flush.fill_(float(i))
+        q2, k2 = q.clone(), k.clone()                        # (warm; the values were last read a launch or a flush ago)
+        out = torch.empty_like(q)
+        a = {**args, "k_packed": k2}
+        if sink:
+            kernels.attention_ext(q2, out, key_dim=d, value_dim=d, sink=sinks, **a)
+        else:
+            kernels.attention(q2, out, head_dim=d, **a)
+        first = out if first is None else first
+        if i % 25 == 24:
+            kernels.check_tc_status()
+            assert torch.equal(out, first)
+    T0 = 200                                                 # and right: the first rows of one sequence by hand
+    rows = slice(3 * L, 3 * L + T0)
+    for h in (0, 5):
+        c = slice(h * d, (h + 1) * d)
+        want = ps.softmax_head(q[rows, c].double().cpu(), k[rows, c].double().cpu(), v[rows, c].double().cpu(), d ** -0.5,
+                               ps.visible(T0), torch.tensor(1.0, dtype=torch.float64) if sink else None)
+        _close(first[rows, c], want, 2e-2, f"head {h}")
+
+
+@pytest.mark.parametrize("H,d", [(4, 64), (2, 128), (3, 32), (2, 96)])
+@pytest.mark.parametrize("window", [None, 70])
+def test_a_gate_per_head_in_the_prompt_kernels(H, d, window):
+    from tq_kv_b200 import kernels
+    T = 150
+    g = torch.Generator().manual_seed(d)
+    q, k, v = (torch.randn(T, H * d, generator=g).to(torch.bfloat16) for _ in range(3))
+    gate = torch.randn(T, H + 3, generator=g)[:, 2:H + 2]
+    sink = torch.randn(H, generator=g)
+    for fast in (True, False):
+        out = torch.empty((T, H * d), dtype=torch.bfloat16, device=DEV)
+        wide = torch.zeros((T, H + 3), device=DEV)
+        wide[:, 2:H + 2] = gate.to(DEV)
+        kernels.attention_ext(q.to(DEV), out, n_heads=H, n_kv_heads=H, key_dim=d, value_dim=d, tok_pos=_ints(list(range(T))),
+                              tok_seq=_ints([0] * T), cu_seqlens=_ints([0, T]), start_pos=_ints([0]), scale=d ** -0.5,
+                              window=window, sink=sink.to(DEV), gate=wide[:, 2:H + 2], k_packed=k.to(DEV), v_packed=v.to(DEV),
+                              use_fast=fast)
+        for h in range(H):
+            c = slice(h * d, (h + 1) * d)
+            want = ps.softmax_head(q[:, c].double(), k[:, c].double(), v[:, c].double(), d ** -0.5, ps.visible(T, window),
+                                   sink[h].double()) * torch.sigmoid(gate[:, h:h + 1].double())
+            _close(out[:, c], want, 2e-2, f"head {h}, fast={fast}")
+
+
+@pytest.mark.parametrize("T,H,d,r,n,row", [(1, 3, 20, 4, 24, 32), (17, 2, 128, 0, 128, 128), (40, 5, 96, 32, 96, 128),
+                                           (64, 1, 130, 2, 200, 208), (5, 4, 12, 6, 10, 32), (33, 2, 64, 64, 512, 576)])
+def test_the_latent_s_per_head_products(T, H, d, r, n, row):
+    """The query into the latent's space and the mean latent out of it, in bfloat16, at sizes around the tensor-core
+    tiles (one whose rows are no whole 16-byte pieces: the general kernel)."""
+    from tq_kv_b200 import kernels
+    g = torch.Generator().manual_seed(T + n)
+    e = d + 3
+    q = torch.randn(T, H * (d + r), generator=g).to(DEV)
+    uk = (torch.randn(H * d, n, generator=g) / d ** 0.5).to(torch.bfloat16).to(DEV)
+    uv = (torch.randn(H * e, n, generator=g) / n ** 0.5).to(torch.bfloat16).to(DEV)
+    pos = torch.arange(T) * 7 + 1
+    rate = torch.pow(torch.tensor(1e4, dtype=torch.float64), -2.0 * torch.arange(max(r // 2, 1), dtype=torch.float64) / max(r, 2))
+    ang = torch.arange(T * 7 + 2, dtype=torch.float64).reshape(-1, 1) * rate
+    qa = torch.full((T, H * row), float("nan"), dtype=torch.bfloat16, device=DEV)
+    kernels.latent_query(q, uk, qa, heads=H, dim=d, rot_dim=r, kv_rank=n, row_width=row, cos=torch.cos(ang).float().to(DEV),
+                         sin=torch.sin(ang).float().to(DEV), rot_dims=r, paired=False, tok_pos=pos.int().to(DEV))
+    Q = q.double().cpu().reshape(T, H, d + r)
+    got = qa.reshape(T, H, row)
+    _close(got[..., :n], torch.einsum("thd,hdn->thn", Q[..., :d], uk.double().cpu().reshape(H, d, n)), 1.5e-2, "query")
+    if r:
+        _close(got[..., n:n + r], ps.rotate(Q[..., d:], pos, r, 1e4), 1e-2, "rotated part")
+    assert not got[..., n + r:].any()
+    lat = torch.randn(T, H * row, generator=g).to(torch.bfloat16).to(DEV)
+    gate = torch.randn(T, H * e, generator=g).to(DEV)
+    y = torch.full((T, H * e), float("nan"), dtype=torch.bfloat16, device=DEV)
+    kernels.latent_expand(lat, uv, y, heads=H, kv_rank=n, row_width=row, value_dim=e, gate=gate)
+    want = torch.einsum("thn,hen->the", lat.double().cpu().reshape(T, H, row)[..., :n], uv.double().cpu().reshape(H, e, n))
+    _close(y.reshape(T, H, e), want * torch.sigmoid(gate.double().cpu().reshape(T, H, e)), 1.5e-2, "expanded")
+
+
 # ---- the latent's kernels without rotation and with a gate per head -------------------------------------------------
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_latent_rows_and_queries_without_a_rotated_part(dtype):

@@ -68,6 +68,7 @@ struct FpOptions {
     const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
     int chunk;              // > 0: keys of the query's own chunk only
     float* out32;           // the result goes here unrounded, [T, nh * HD] (`out` is then not used); or null
+    int head_gate;          // the gate is one number per head (column h) instead of one per entry
 };
 
 // cap * tanh(x / cap) with 2^x and a fast division (a few ulp; tanh.approx is not enough)
@@ -292,9 +293,11 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
     for (int r = 0; r < 2; ++r) {
         if (ri[r] >= len) continue;
         // (the sink's share of the denominator is 2^(sink log2 e - m) in the units the sums are kept in)
-        const float inv = 1.f / ((EXT && opt.sinks) ? l_run[r] + exp2f(fmaf(opt.sinks[h], 1.4426950408889634f, -m_run[r])) : l_run[r]);
+        float inv = 1.f / ((EXT && opt.sinks) ? l_run[r] + exp2f(fmaf(opt.sinks[h], 1.4426950408889634f, -m_run[r])) : l_run[r]);
         bf16* orow = out + ((size_t)(tok0 + ri[r]) * nh + h) * HD;
-        const float* grow = (EXT && opt.gate) ? opt.gate + (size_t)(tok0 + ri[r]) * opt.ldg + (size_t)h * HD : nullptr;
+        if (EXT && opt.gate && opt.head_gate)
+            inv *= 1.f / (1.f + expf(-opt.gate[(size_t)(tok0 + ri[r]) * opt.ldg + h]));
+        const float* grow = (EXT && opt.gate && !opt.head_gate) ? opt.gate + (size_t)(tok0 + ri[r]) * opt.ldg + (size_t)h * HD : nullptr;
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
             const int d = n * 8 + 2 * tid4;
@@ -314,7 +317,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, FpSource src, const int* __rest
 template <int HD, bool EXT = false>
 static int launch_flash_prefill(const bf16* q, const FpSource& src, const int* cu_seqlens, const int* start_pos,
                                 int n_seqs, int n_tokens, int window, float scale, bf16* out, int nh, int nkv,
-                                cudaStream_t stream, FpOptions opt = FpOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0, nullptr}) {
+                                cudaStream_t stream, FpOptions opt = FpOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0, nullptr, 0}) {
     constexpr size_t smem = 2 * 2 * FP_BN * (HD * 2 + 16);
     static bool configured = false;
     if (!configured) {
@@ -362,7 +365,7 @@ TQ_API int tq_flash_prefill_ext(const void* q, const void* k_packed, const void*
                                 const void* v_pages, const int* block_table, int table_width, int ring_pages,
                                 int page_tokens, const int* cu_seqlens, const int* start_pos, int n_seqs, int n_tokens,
                                 int window, float scale, float softcap, const float* slopes, int keep_first,
-                                const float* sinks, int chunk, const float* gate, int ldg, void* out, int out_f32, int nh,
+                                const float* sinks, int chunk, const float* gate, int ldg, int head_gate, void* out, int out_f32, int nh,
                                 int nkv, int hd, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (nkv <= 0 || nh % nkv || nh > 65535) return (int)cudaErrorNotSupported;
@@ -371,7 +374,7 @@ TQ_API int tq_flash_prefill_ext(const void* q, const void* k_packed, const void*
     FpSource src{(const bf16*)k_packed, (const bf16*)v_packed, (const bf16*)k_pages, (const bf16*)v_pages,
                  block_table, table_width, ring_pages, page_tokens};
     if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
-    const FpOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk, out_f32 ? (float*)out : nullptr};
+    const FpOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk, out_f32 ? (float*)out : nullptr, head_gate};
 #define TQ_FP(H)                                                                                                    \
     case H:                                                                                                         \
         return launch_flash_prefill<H, true>((const bf16*)q, src, cu_seqlens, start_pos, n_seqs, n_tokens, window, \

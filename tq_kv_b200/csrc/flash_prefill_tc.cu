@@ -31,13 +31,15 @@
 //
 // Order between the threads, beyond the producer/consumer pairs: the MMA
 // thread waits for the P·V of the tile before (p_empty) before it issues the
-// Q·K^T of the tile after, which writes over that tile's P; a softmax thread
-// waits for the phase of p_full before its own before it arrives again (it may
-// be a whole tile ahead of the slowest thread, and a second arrival in the
-// same phase would stand in for the slow thread's first); the end of the last
-// P·V has a barrier of its own (o_done), since the softmax threads follow
-// p_empty only when they rescale O and a wait by parity cannot tell a phase
-// that is two behind from one that is done.  Two load tests guard this.
+// Q·K^T of the tile after, which writes over that tile's P; p_full is one
+// barrier per score buffer: the softmax threads may finish two tiles before
+// the MMA thread, held up by a V tile that is late, looks at the first, and a
+// wait by parity cannot tell a phase that is two behind from one that is
+// still open (with one barrier for all tiles such a block waited for good).
+// They cannot come back to the same buffer before that tile's P·V is done,
+// which also keeps a fast thread's arrival out of a slow thread's phase; the
+// end of the last P·V has a barrier of its own (o_done) for the same reason.
+// Load tests guard this.
 //
 // Formulas: src/models/turbo_generic.rs:1620-1631 (see attention.cu).
 #include <cuda.h>
@@ -176,6 +178,7 @@ struct FtOptions {
     const float* sinks;     // [nh] or null: exp(sinks[h]) added to the softmax's denominator (a key without a value)
     int chunk;              // > 0: keys of the query's own chunk only
     float* out32;           // the result goes here unrounded, [T, nh * HD] (`out` is then not used); or null
+    int head_gate;          // the gate is one number per head (column h) instead of one per entry
 };
 
 template <int HD, bool PAGED, int WEIGHTS>
@@ -206,10 +209,10 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     uint64_t* v_full = bars + 5;                           // [2]  the tile's P·V, so the load of the tile after
     uint64_t* v_empty = bars + 7;                          // [2]  next has a whole iteration to arrive
     uint64_t* s_full = bars + 9;                           // [2]
-    uint64_t* p_full = bars + 11;                          // 128 arrivals (softmax threads)
-    uint64_t* p_empty = bars + 12;                         // the P·V of a tile is done: O may be touched
-    uint64_t* o_done = bars + 13;                          // once: the last P·V is done, O is final
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
+    uint64_t* p_full = bars + 11;                          // [2]  128 arrivals (softmax threads)
+    uint64_t* p_empty = bars + 13;                         // the P·V of a tile is done: O may be touched
+    uint64_t* o_done = bars + 14;                          // once: the last P·V is done, O is final
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
     volatile uint32_t* failed = tmem_slot + 1;
 
     // which (sequence, 128-token tile) is this block's?  Later tiles of a sequence have more keys to walk:
@@ -250,8 +253,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(ft_smem(&v_full[s])));
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(ft_smem(&v_empty[s])));
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(ft_smem(&s_full[s])));
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], 128;\n" ::"r"(ft_smem(&p_full[s])));
         }
-        asm volatile("mbarrier.init.shared::cta.b64 [%0], 128;\n" ::"r"(ft_smem(p_full)));
         asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(ft_smem(p_empty)));
         asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(ft_smem(o_done)));
         *failed = 0;
@@ -336,7 +339,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                 // relies on.
                 if (it > 0 && !ft_wait(ft_smem(p_empty), (it - 1) & 1)) { *failed = 1; ok = false; break; }
                 if (it + 1 < n_tiles && !issue_qk(it + 1)) { *failed = 1; ok = false; break; }
-                if (!ft_wait(ft_smem(&v_full[s]), (it >> 1) & 1) || !ft_wait(ft_smem(p_full), it & 1)) {
+                if (!ft_wait(ft_smem(&v_full[s]), (it >> 1) & 1) || !ft_wait(ft_smem(&p_full[s]), (it >> 1) & 1)) {
                     *failed = 1; ok = false; break;
                 }
                 asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
@@ -366,11 +369,13 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         const bool ext_capped = WEIGHTS == FT_SOFTMAX_EXT && opt.softcap > 0.f;
         const float ext_in = WEIGHTS != FT_SOFTMAX_EXT ? 0.f
             : (ext_capped ? opt.scale * (2.f * 1.4426950408889634f / opt.softcap) : opt.scale * 1.4426950408889634f);
+        // neither a cap nor slopes: the scores stay as they are and the scale rides in the exponent, as without options
+        const bool ext_plain = WEIGHTS == FT_SOFTMAX_EXT && !ext_capped && !opt.slopes;
         const float ext_cap = ext_capped ? opt.softcap * 1.4426950408889634f : 0.f;
         const float ext_slope = (WEIGHTS == FT_SOFTMAX_EXT && opt.slopes) ? opt.slopes[h] * 1.4426950408889634f : 0.f;
         if constexpr (WEIGHTS == FT_SOFTMAX_EXT) {
             // the row's gate values are wanted when O leaves: ask L2 for them now (lines of 32 floats)
-            if (opt.gate) {
+            if (opt.gate && !opt.head_gate) {
                 const float* gp = opt.gate + (size_t)(tok0 + min(i_row, len - 1)) * opt.ldg + (size_t)h * HD;
                 for (int c = 0; c < HD; c += 32) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(gp + c));
                 asm volatile("prefetch.global.L2 [%0];\n" ::"l"(gp + HD - 1));
@@ -412,7 +417,15 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                     }
                     return fmaf(-ext_slope, d0 - (float)j, x);
                 };
-                if (inside) {
+                if (ext_plain) {
+                    if (!inside) {
+#pragma unroll
+                        for (int j = 0; j < FT_BN; ++j) {
+                            const int key = j0 + j;
+                            if (key > j_hi || (key < j_lo && key >= keep)) sv[j] = -INFINITY;
+                        }
+                    }
+                } else if (inside) {
 #pragma unroll
                     for (int j = 0; j < FT_BN; ++j) sv[j] = weigh(sv[j], j);
                 } else {
@@ -445,9 +458,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                     packed[j >> 1] = __uint_as_float(*reinterpret_cast<uint32_t*>(&pk));
                 }
                 ft_st32(s_addr, packed);
-                if (it > 0 && !ft_wait(ft_smem(p_full), (it - 1) & 1, true)) { *failed = 1; ok = false; break; }
                 asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
-                ft_arrive(ft_smem(p_full));
+                ft_arrive(ft_smem(&p_full[it & 1]));
                 continue;
             }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};    // four chains instead of one of 64
@@ -459,7 +471,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                 mx4[3] = fmaxf(mx4[3], sv[j + 3]);
             }
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const float sl = WEIGHTS == FT_SOFTMAX_EXT ? 1.f : scale_log2;      // EXT: already in units of log2
+            const float sl = WEIGHTS == FT_SOFTMAX_EXT && !ext_plain ? 1.f : scale_log2;      // EXT: already in units of log2
             const float m_tile = mx * sl;
             const bool grow = m_tile > m_ref + 8.f;          // also true for the first finite maximum
             if (__any_sync(0xffffffffu, grow) && it > 0) {
@@ -497,19 +509,16 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             }
             ft_st32(s_addr, packed);
             l_run += (rs4[0] + rs4[1]) + (rs4[2] + rs4[3]);
-            // A thread that is a whole tile ahead of the slowest must not arrive again before the phase of the
-            // tile before is complete: its second arrival would stand in for the slow thread's first, and the
-            // P·V would start without that thread's rows of P.  (While P went through shared memory, waiting for
-            // the P·V of the tile before kept the threads together.)
-            if (it > 0 && !ft_wait(ft_smem(p_full), (it - 1) & 1, true)) { *failed = 1; ok = false; break; }
+            // (The next arrival on this barrier is two tiles on: those scores are issued only after this tile's P·V,
+            // so no thread can arrive twice in one phase, nor can the MMA thread miss a phase.)
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
-            ft_arrive(ft_smem(p_full));
+            ft_arrive(ft_smem(&p_full[it & 1]));
         }
         // The last tile's P·V, then O / l.  (A barrier of its own: the softmax threads no longer follow every
         // phase of p_empty, and a wait by parity cannot tell a phase that is two behind from one that is done.)
         // The gate's values of the row come in pieces of 32, each loaded while the piece before is applied; the
         // first is asked for before the wait for the last P·V.
-        const float* grow = (WEIGHTS == FT_SOFTMAX_EXT && opt.gate)
+        const float* grow = (WEIGHTS == FT_SOFTMAX_EXT && opt.gate && !opt.head_gate)
                                 ? opt.gate + (size_t)(tok0 + min(i_row, len - 1)) * opt.ldg + (size_t)h * HD : nullptr;
         float4 g_next[8];
         if (WEIGHTS == FT_SOFTMAX_EXT && grow) {
@@ -522,6 +531,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             float inv = 1.f / l_run;
             if constexpr (WEIGHTS == FT_SOFTMAX_EXT) {         // the sink's share: 2^(sink log2 e - m_ref), the sums' unit
                 if (opt.sinks) inv = 1.f / (l_run + exp2f(fmaf(opt.sinks[h], 1.4426950408889634f, -m_ref)));
+                if (opt.gate && opt.head_gate)
+                    inv *= 1.f / (1.f + expf(-opt.gate[(size_t)(tok0 + min(i_row, len - 1)) * opt.ldg + h]));
             }
             if constexpr (WEIGHTS == FT_SIGMOID)
                 inv = gate ? 1.f / (1.f + expf(-gate[(size_t)(tok0 + min(i_row, len - 1)) * ldg + h])) : 1.f;
@@ -595,7 +606,7 @@ static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
                      int table_width, int ring_pages, const int* cu_seqlens, const int* start_pos, int n_seqs,
                      int n_tokens, int window, float scale, bf16* out, int nh, int nkv, int* status,
                      cudaStream_t stream, const float* bias = nullptr, int n_dist = 0, const float* gate = nullptr,
-                     int ldg = 0, FtOptions opt = FtOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0, nullptr}) {
+                     int ldg = 0, FtOptions opt = FtOptions{0.f, 0.f, nullptr, 0, nullptr, 0, nullptr, 0, nullptr, 0}) {
     constexpr int SMEM = (HD / 64) * (FT_SUB_BYTES + 4 * FT_KV_SUB_BYTES) + 256;
     static bool configured = false;
     if (!configured) {
@@ -688,7 +699,7 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
                                    int ring_pages, int page_tokens, const int* cu_seqlens, const int* start_pos,
                                    int n_seqs, int n_tokens, int window, float scale, float softcap,
                                    const float* slopes, int keep_first, const float* sinks, int chunk,
-                                   const float* gate, int ldg, void* out, int out_f32, int nh,
+                                   const float* gate, int ldg, int head_gate, void* out, int out_f32, int nh,
                                    int nkv, int hd, int* status, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (nkv <= 0 || nh % nkv || (hd != 64 && hd != 128)) return (int)cudaErrorNotSupported;
@@ -696,7 +707,7 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
     const bool paged = k_packed == nullptr;
     if (paged && (page_tokens != 64 || !k_pages || !v_pages || !block_table)) return (int)cudaErrorNotSupported;
     if (keep_first < 0 || (keep_first > 0 && paged && ring_pages > 0)) return (int)cudaErrorInvalidValue;
-    if (gate && ((ldg & 3) || (reinterpret_cast<uintptr_t>(gate) & 15))) return (int)cudaErrorNotSupported;
+    if (gate && !head_gate && ((ldg & 3) || (reinterpret_cast<uintptr_t>(gate) & 15))) return (int)cudaErrorNotSupported;
     CUtensorMap mq, mk, mv;
     int st = ft_map(&mq, q, (uint64_t)n_tokens, (uint64_t)nh * hd, (uint64_t)nh * hd, FT_BM);
     if (st) return st;
@@ -709,7 +720,7 @@ TQ_API int tq_flash_prefill_tc_ext(const void* q, const void* k_packed, const vo
     }
     if (st) return st;
     if (chunk < 0 || (chunk > 0 && window > 0)) return (int)cudaErrorInvalidValue;
-    const FtOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk, out_f32 ? (float*)out : nullptr};
+    const FtOptions opt{scale, softcap, slopes, keep_first, gate, ldg, sinks, chunk, out_f32 ? (float*)out : nullptr, head_gate};
 #define TQ_FT(H, P) return ft_launch<H, P, FT_SOFTMAX_EXT>(mq, mk, mv, block_table, table_width, ring_pages, cu_seqlens, \
                                                            start_pos, n_seqs, n_tokens, window, scale, (bf16*)out, nh,    \
                                                            nkv, status, stream, nullptr, 0, nullptr, 0, opt)

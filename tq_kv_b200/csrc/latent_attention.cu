@@ -16,6 +16,8 @@
 //   latent_expand  per (token, head): o[h] = U_v[h] mean(c), times sigmoid(gate) entry by entry or (head_gate) with one
 //                  gate per head
 //
+// In bfloat16 latent_query and latent_expand run on the tensor cores (latent_product_kernel), 16 tokens at a time.
+//
 //   latent_heads   for prompts that bring all their keys along: per (token, head) the query [q_flat, rot(q_rot), 0 ...],
 //                  the expanded key [U_k[h] c, k_r, 0 ...] and the value [U_v[h] c, 0 ...], all `hw` wide, for the
 //                  ordinary attention kernels (whose heads then are this mixer's heads); latent_expand without a
@@ -148,6 +150,51 @@ __global__ void latent_heads_kernel(const float* __restrict__ q, int ldq, const 
     }
 }
 
+// The same for bfloat16 with d, r, e and hw in multiples of four and aligned rows: a block per token, a thread per four
+// neighbouring entries of a head's q, k and v.
+__device__ __forceinline__ void lh_store4(bf16* dst, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+__global__ void __launch_bounds__(256)
+latent_heads4_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ kfv, int ldk, int off_v,
+                     const bf16* __restrict__ rows, int rp, int n, int H, int d, int r, int e, int hw,
+                     const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims, int paired,
+                     const int* __restrict__ tok_pos, bf16* __restrict__ q_out, bf16* __restrict__ k_out,
+                     bf16* __restrict__ v_out) {
+    const int t = blockIdx.x, hw4 = hw >> 2;
+    pdl_wait();
+    pdl_launch();
+    const size_t at = (size_t)tok_pos[t] * (rot_dims >> 1);
+    const float *cs = cos_t + at, *sn = sin_t + at;
+    const float* qt = q + (size_t)t * ldq;
+    const float* kt = kfv + (size_t)t * ldk;
+    const bf16* rr = rows + (size_t)t * rp + n;
+    const uint2 none = make_uint2(0u, 0u);
+    for (int p = threadIdx.x; p < H * hw4; p += blockDim.x) {
+        const int h = p / hw4, i = (p - h * hw4) * 4;
+        const size_t o = ((size_t)t * H + h) * hw + i;
+        const float* qr = qt + h * (d + r);
+        if (i < d) {
+            lh_store4(q_out + o, *reinterpret_cast<const float4*>(qr + i));
+            lh_store4(k_out + o, *reinterpret_cast<const float4*>(kt + h * d + i));
+        } else if (i < d + r) {
+            float4 v;
+            v.x = rot_entry(qr + d, i - d, rot_dims, paired, cs, sn);
+            v.y = rot_entry(qr + d, i - d + 1, rot_dims, paired, cs, sn);
+            v.z = rot_entry(qr + d, i - d + 2, rot_dims, paired, cs, sn);
+            v.w = rot_entry(qr + d, i - d + 3, rot_dims, paired, cs, sn);
+            lh_store4(q_out + o, v);
+            *reinterpret_cast<uint2*>(k_out + o) = *reinterpret_cast<const uint2*>(rr + i - d);
+        } else {
+            *reinterpret_cast<uint2*>(q_out + o) = none;
+            *reinterpret_cast<uint2*>(k_out + o) = none;
+        }
+        if (i < e) lh_store4(v_out + o, *reinterpret_cast<const float4*>(kt + off_v + h * e + i));
+        else *reinterpret_cast<uint2*>(v_out + o) = none;
+    }
+}
+
 template <typename T>
 __global__ void latent_expand_kernel(const T* __restrict__ lat, int H, int n, int rp, int e, const T* __restrict__ uv,
                                      const float* __restrict__ gate, int ldg, int head_gate, T* __restrict__ out) {
@@ -181,6 +228,124 @@ __global__ void latent_expand_kernel(const T* __restrict__ lat, int H, int n, in
     }
 }
 
+// ---- the per-head products on the tensor cores (bfloat16) ------------------------------------------------------------
+// C[t, h, :N] = A[t, h, :K] . B_h for 16 tokens and 64 columns of one head per block: the head's matrix is read once
+// per 16 tokens instead of once per token.  KN: B_h lies [K, N] (latent_query: U_k[h], k rows of n entries), else
+// [N, K] (latent_expand: U_v[h], e rows of n entries); both with rows of whole 16-byte pieces.  A (float32 queries or
+// bfloat16 means) is rounded to bfloat16 in shared memory, sums are float32; K is walked in pieces of LP_KC.
+// The epilogue rounds once: for queries the first column tile also writes the rotated part and the row's padding; for
+// results the gate is applied.
+#define LP_TOK 16
+#define LP_COLS 64
+#define LP_KC 128
+
+__device__ __forceinline__ void lp_ldmatrix_x4(uint32_t* r, const void* smem) {
+    const uint32_t addr = (uint32_t)__cvta_generic_to_shared(smem);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void lp_ldmatrix_x4_trans(uint32_t* r, const void* smem) {
+    const uint32_t addr = (uint32_t)__cvta_generic_to_shared(smem);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void lp_mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+struct LpQuery {          // what the query's epilogue needs beyond the product
+    int d, r, rp, rot_dims, paired;
+    const float *cos_t, *sin_t;
+    const int* tok_pos;
+};
+
+template <typename TA, bool KN>
+__global__ void __launch_bounds__(128)
+latent_product_kernel(const TA* __restrict__ a, int lda, int a_head, const bf16* __restrict__ w, int H, int K, int N,
+                      bf16* __restrict__ out, int out_head, int n_tokens, LpQuery qq, const float* __restrict__ gate,
+                      int ldg, int head_gate) {
+    constexpr int AW = LP_KC + 8;                              // padded rows: ldmatrix without bank conflicts
+    constexpr int BW = KN ? LP_COLS + 8 : LP_KC + 8;
+    constexpr int BROWS = KN ? LP_KC : LP_COLS;
+    __shared__ __align__(16) bf16 a_s[LP_TOK * AW];
+    __shared__ __align__(16) bf16 b_s[BROWS * BW];
+    const int h = blockIdx.x, c0 = blockIdx.y * LP_COLS, t0 = blockIdx.z * LP_TOK;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const bf16 zero = __float2bfloat16_rn(0.f);
+    const bf16* wh = w + (size_t)h * K * N;
+    // the first piece of the head's matrix does not depend on the kernel before
+    auto load_b = [&](int k0) {
+        for (int p = threadIdx.x; p < BROWS * (KN ? LP_COLS : LP_KC) / 8; p += 128) {
+            const int per = (KN ? LP_COLS : LP_KC) / 8;
+            const int row = p / per, c = (p - row * per) * 8;
+            const int k = KN ? k0 + row : k0 + c, n = KN ? c0 + c : c0 + row;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (k < K && n < N) v = *reinterpret_cast<const uint4*>(wh + (KN ? (size_t)k * N + n : (size_t)n * K + k));
+            *reinterpret_cast<uint4*>(b_s + row * BW + c) = v;
+        }
+    };
+    load_b(0);
+    pdl_wait();
+    pdl_launch();
+    float acc[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
+    for (int k0 = 0; k0 < K; k0 += LP_KC) {
+        const int kc = min(LP_KC, (K - k0 + 15) & ~15);
+        if (k0 > 0) { __syncthreads(); load_b(k0); }
+        for (int p = threadIdx.x; p < LP_TOK * LP_KC / 2; p += 128) {
+            const int row = p / (LP_KC / 2), c = (p - row * (LP_KC / 2)) * 2, t = t0 + row, k = k0 + c;
+            bf16 v0 = zero, v1 = zero;
+            if (t < n_tokens) {
+                const TA* ar = a + (size_t)t * lda + (size_t)h * a_head;
+                if (k < K) v0 = from_f32<bf16>(to_f32<TA>(ar[k]));
+                if (k + 1 < K) v1 = from_f32<bf16>(to_f32<TA>(ar[k + 1]));
+            }
+            a_s[row * AW + c] = v0;
+            a_s[row * AW + c + 1] = v1;
+        }
+        __syncthreads();
+        const int mat = lane >> 3, r8 = lane & 7;
+        for (int ks = 0; ks < kc; ks += 16) {
+            uint32_t af[4], bfr[4];
+            lp_ldmatrix_x4(af, a_s + ((mat & 1) * 8 + r8) * AW + ks + (mat >> 1) * 8);
+            if (KN) lp_ldmatrix_x4_trans(bfr, b_s + (ks + (mat & 1) * 8 + r8) * BW + warp * 16 + (mat >> 1) * 8);
+            else lp_ldmatrix_x4(bfr, b_s + (warp * 16 + (mat >> 1) * 8 + r8) * BW + ks + (mat & 1) * 8);
+            lp_mma(acc[0], af, bfr[0], bfr[1]);
+            lp_mma(acc[1], af, bfr[2], bfr[3]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int t = t0 + (lane >> 2) + 8 * (e >> 1), n = c0 + warp * 16 + i * 8 + 2 * (lane & 3) + (e & 1);
+            if (t < n_tokens && n < N) {
+                float v = acc[i][e];
+                if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + (head_gate ? h : h * N + n)]));
+                out[((size_t)t * H + h) * out_head + n] = from_f32<bf16>(v);
+            }
+        }
+    if (KN && blockIdx.y == 0) {                               // the rotated part and the padding behind it
+        const int rest = qq.rp - N;
+        for (int p = threadIdx.x; p < LP_TOK * rest; p += 128) {
+            const int row = p / rest, i = p - row * rest, t = t0 + row;
+            if (t >= n_tokens) continue;
+            float v = 0.f;
+            if (i < qq.r) {
+                const size_t at = (size_t)qq.tok_pos[t] * (qq.rot_dims >> 1);
+                const TA* ar = a + (size_t)t * lda + (size_t)h * a_head + qq.d;
+                if constexpr (sizeof(TA) == 4) v = rot_entry(ar, i, qq.rot_dims, qq.paired, qq.cos_t + at, qq.sin_t + at);
+            }
+            out[((size_t)t * H + h) * out_head + N + i] = from_f32<bf16>(v);
+        }
+    }
+}
+
+static bool lp_aligned(const void* p, int row) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && row % 8 == 0; }
+
 TQ_API int tq_latent_rows(const float* proj, int ld, int off_q, int off_kv, int q_rank, int n, int r, int rp,
                           const float* wq, const float* wkv, float eps, const float* cos_t, const float* sin_t,
                           int rot_dims, int paired, const int* tok_pos, const int* tok_seq, const int* new_lens,
@@ -213,6 +378,11 @@ TQ_API int tq_latent_query(const float* q, int ldq, int H, int d, int r, int n, 
     if (!q || !uk || !cos_t || !sin_t || !tok_pos || !out || H <= 0 || H > 65535 || d <= 0 || r < 0 || n <= 0 ||
         rp < n + r || rot_dims < 0 || rot_dims > r || (rot_dims & 1))
         return (int)cudaErrorInvalidValue;
+    if (dtype == TQ_BF16 && lp_aligned(uk, n) && (n_tokens + LP_TOK - 1) / LP_TOK <= 65535 && (n + LP_COLS - 1) / LP_COLS <= 65535)
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_product_kernel<float, true>,
+                             dim3(H, (n + LP_COLS - 1) / LP_COLS, (n_tokens + LP_TOK - 1) / LP_TOK), dim3(128), 0, stream, q,
+                             ldq, d + r, (const bf16*)uk, H, d, n, (bf16*)out, rp, n_tokens,
+                             LpQuery{d, r, rp, rot_dims, paired, cos_t, sin_t, tok_pos}, (const float*)nullptr, 0, 0);
     const int threads = rp > 128 ? 256 : 128;
     const size_t smem = (size_t)(d + r) * sizeof(float);
     const dim3 grid(n_tokens, H);
@@ -229,6 +399,12 @@ TQ_API int tq_latent_expand(const void* lat, int H, int n, int rp, int e, const 
                             int head_gate, void* out, int dtype, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (!lat || !out || H <= 0 || H > 65535 || n <= 0 || rp < n || e <= 0 || (!uv && e > n)) return (int)cudaErrorInvalidValue;
+    if (dtype == TQ_BF16 && uv && lp_aligned(uv, n) && (n_tokens + LP_TOK - 1) / LP_TOK <= 65535 &&
+        (e + LP_COLS - 1) / LP_COLS <= 65535)
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_product_kernel<bf16, false>,
+                             dim3(H, (e + LP_COLS - 1) / LP_COLS, (n_tokens + LP_TOK - 1) / LP_TOK), dim3(128), 0, stream,
+                             (const bf16*)lat, H * rp, rp, (const bf16*)uv, H, n, e, (bf16*)out, e, n_tokens,
+                             LpQuery{0, 0, 0, 0, 0, nullptr, nullptr, nullptr}, gate, ldg, head_gate);
     const size_t smem = (size_t)n * sizeof(float);
     const dim3 grid(n_tokens, H);
     if (dtype == TQ_F32)
@@ -248,6 +424,12 @@ TQ_API int tq_latent_heads(const float* q, int ldq, const float* kfv, int ldk, i
     if (!q || !kfv || !rows || !cos_t || !sin_t || !tok_pos || !q_out || !k_out || !v_out || H <= 0 || H > 65535 ||
         d <= 0 || r < 0 || e <= 0 || hw < d + r || hw < e || rp < n + r || rot_dims < 0 || rot_dims > r || (rot_dims & 1))
         return (int)cudaErrorInvalidValue;
+    auto al = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+    if (dtype == TQ_BF16 && !((d | r | e | hw | n | ldq | ldk | off_v) & 3) && !(rp & 3) && al(q, 16) && al(kfv, 16) &&
+        al(rows, 8) && al(q_out, 8) && al(k_out, 8) && al(v_out, 8))
+        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_heads4_kernel, dim3(n_tokens), dim3(256), 0, stream, q, ldq, kfv, ldk,
+                             off_v, (const bf16*)rows, rp, n, H, d, r, e, hw, cos_t, sin_t, rot_dims, paired, tok_pos,
+                             (bf16*)q_out, (bf16*)k_out, (bf16*)v_out);
     const dim3 grid(n_tokens, H);
     const size_t smem = (size_t)(r > 0 ? r : 1) * sizeof(float);
     if (dtype == TQ_F32)

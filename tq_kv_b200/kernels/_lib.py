@@ -225,11 +225,11 @@ _SIGNATURES = {
                          c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
     "tq_flash_prefill_tc_ext": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int,
                                 c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p,
-                                c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+                                c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
                                 c_void_p],
     "tq_flash_prefill_ext": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                              c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p,
-                             c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                             c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "tq_flash_decode_ext": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                             c_float, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                             c_int, c_int, c_void_p],

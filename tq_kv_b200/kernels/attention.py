@@ -146,7 +146,8 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
     i // chunk == j // chunk.  `sink`: a float32 tensor [n_heads] — the softmax's denominator counts one more key of
     score sink[h] that has no value, p_j = exp(s_j) / (exp(sink[h]) + sum exp(s)) — or True (a score of 0) or False.
     Value rows may have another width than the keys.  q [T, nh*key_dim], out [T, nh*value_dim]; keys and values as in `attention`.
-    `gate` (float32 [T, nh*value_dim], possibly a column slice of wider rows): out *= sigmoid(gate), in the
+    `gate` (float32 [T, nh*value_dim], or [T, nh] with one number per head, possibly a column slice of wider rows): out
+    *= sigmoid(gate), in the
     attention kernel's last step where it can, else by a kernel of its own.
     `unmerged` (then `out` is None; no gate, no sink): the float32 results are returned for a kernel that goes on with
     them, (rows [T, nh, value_dim], None, 1) or, per split of the keys, (sums [T, nh, n, value_dim], their maxima and
@@ -196,14 +197,15 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
         part_acc, part_ml = scratch[:n_acc], scratch[n_acc:need]
     need_contiguous(q=q, out=out, k_packed=k_packed, v_packed=v_packed, k_pages=k_pages, v_pages=v_pages,
                     block_table=block_table, slopes=slopes, sink=sink)
-    if gate is not None and (gate.dtype != torch.float32 or tuple(gate.shape) != tuple(out.shape)
-                             or gate.stride(1) != 1):
-        raise KernelError("attention: the gate must be float32 of the result's shape")
+    if gate is not None and (gate.dtype != torch.float32 or tuple(gate.shape) not in (tuple(out.shape), (T, n_heads))
+                             or (gate.stride(1) != 1 and gate.shape[1] > 1)):
+        raise KernelError("attention: the gate must be float32 of the result's shape, or one number per head")
+    head_gate = int(gate is not None and tuple(gate.shape) != tuple(out.shape))
     keep = int(keep_first) if window else 0
     n_seqs = cu_seqlens.shape[0] - 1
     fast = use_fast and q.dtype == torch.bfloat16 and key_dim == value_dim
     if fast and T > n_seqs:                                  # prompts (some sequence brings several tokens)
-        gate_ok = gate is not None and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0
+        gate_ok = gate is not None and (head_gate or (gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0))
         g_ptr, g_ld = (ptr(gate), gate.stride(0)) if gate_ok else (None, 0)
         st = NOT_SUPPORTED
         if USE_TC_ATTENTION:
@@ -211,7 +213,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
                 ptr(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages),
                 0 if k_pages is None else k_pages.shape[0], ptr(block_table), table_width, ring_pages, page_tokens,
                 ptr(cu_seqlens), ptr(start_pos), n_seqs, T, int(window or 0), float(scale), float(softcap or 0.0),
-                ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, ptr(part_acc if unmerged else out),
+                ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, head_gate, ptr(part_acc if unmerged else out),
                 int(unmerged), n_heads, n_kv_heads, key_dim, ptr(tc_status_word(q.device)), stream())
             if st != NOT_SUPPORTED:
                 check(st, "flash_prefill_tc_ext")
@@ -219,7 +221,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, *, n_heads: int, n_kv_head
             st = core().tq_flash_prefill_ext(
                 ptr(q), ptr(k_packed), ptr(v_packed), ptr(k_pages), ptr(v_pages), ptr(block_table), table_width,
                 ring_pages, page_tokens, ptr(cu_seqlens), ptr(start_pos), n_seqs, T, int(window or 0), float(scale),
-                float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld,
+                float(softcap or 0.0), ptr(slopes), keep, ptr(sink), int(chunk or 0), g_ptr, g_ld, head_gate,
                 ptr(part_acc if unmerged else out), int(unmerged), n_heads, n_kv_heads, key_dim, stream())
             if st != NOT_SUPPORTED:
                 check(st, "flash_prefill_ext")

@@ -368,7 +368,8 @@ def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor):
     """x[t, i] *= sigmoid(gate[t, i]) in place, or with fewer gates than entries (one per head) sigmoid(gate[t, i // (n /
     gates)]); gate float32, possibly a column slice of wider rows."""
     T, n = x.shape
-    if gate.dtype != torch.float32 or gate.shape[0] != T or n % gate.shape[1] or gate.stride(1) != 1 or not x.is_contiguous():
+    if gate.dtype != torch.float32 or gate.shape[0] != T or n % gate.shape[1] \
+            or (gate.stride(1) != 1 and gate.shape[1] > 1) or not x.is_contiguous():
         raise KernelError("sigmoid_gate: gate must be float32 [T, n] or [T, heads], x contiguous")
     check(core().tq_sigmoid_gate(ptr(x), dtype_code(x), ptr(gate), gate.stride(0), T, n, n // gate.shape[1], stream()),
           "sigmoid_gate")

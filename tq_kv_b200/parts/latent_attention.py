@@ -132,6 +132,7 @@ class LatentAttention(Mixer):
         self.head_width = -(-need // 16) * 16
         if act == torch.bfloat16:
             self.head_width = next((w for w in kernels.TENSOR_CORE_WIDTHS if w >= need), self.head_width)
+        self.plain_heads = bool(self.q_rank) and not self.rot_dim and self.dim == self.value_dim == self.head_width
         self.w_o = tensors[self._n("out")].contiguous()
         self.q_norm_w = float32_vector(tensors[self._n("q_norm")]) if self.q_rank else None
         self.kv_norm_w = float32_vector(tensors[self._n("kv_norm")]) if not self.shared_kv else None
@@ -191,7 +192,7 @@ class LatentAttention(Mixer):
                                 ring_pages=kv.ring_pages if owns else 0, out_dtype=act, **rot)
             kernels.mark("rotary")
         if self.q_rank:
-            q = kernels.linear(cq, self.w_uq, out_dtype=torch.float32)
+            q = kernels.linear(cq, self.w_uq, out_dtype=act if packed and self.plain_heads else torch.float32)
             kernels.mark("qkv")
         else:
             q = proj[:, :self.q_cols]
@@ -203,18 +204,30 @@ class LatentAttention(Mixer):
             # A prompt from position 0 brings all its keys along: they are expanded once (two matrix products for
             # all heads) and the ordinary attention kernels run with this mixer's heads as they are.
             hw = self.head_width
-            kfv = kernels.linear(rows[:, :self.kv_rank], self.w_ukv, out_dtype=torch.float32)
-            kernels.mark("qkv")
-            qh, kh, vh = (torch.empty((T, H * hw), dtype=act, device=dev) for _ in range(3))
-            kernels.latent_heads(q, kfv, rows, qh, kh, vh, heads=H, dim=self.dim, rot_dim=self.rot_dim,
-                                 value_dim=self.value_dim, kv_rank=self.kv_rank, **rot)
-            kernels.mark("rotary")
-            oh = torch.empty_like(qh)
-            self._attend(qh, oh, hw, k_packed=kh, v_packed=vh, n_kv_heads=H, **common)
-            kernels.mark("attention")
-            kernels.latent_expand(oh, None, y, heads=H, kv_rank=hw, row_width=hw, value_dim=self.value_dim, gate=gate,
-                                  head_gate=self.head_gate)
-            kernels.mark("rotary")
+            lat = rows[:, :self.kv_rank]
+            if self.plain_heads:
+                # nothing to turn and nothing to fill up: the products leave the heads as the attention takes them
+                qh = q
+                kh = kernels.linear(lat, self.w_uk, out_dtype=act)
+                vh = kernels.linear(lat, self.w_uv, out_dtype=act)
+                kernels.mark("qkv")
+            else:
+                kfv = kernels.linear(lat, self.w_ukv, out_dtype=torch.float32)
+                kernels.mark("qkv")
+                qh, kh, vh = (torch.empty((T, H * hw), dtype=act, device=dev) for _ in range(3))
+                kernels.latent_heads(q, kfv, rows, qh, kh, vh, heads=H, dim=self.dim, rot_dim=self.rot_dim,
+                                     value_dim=self.value_dim, kv_rank=self.kv_rank, **rot)
+                kernels.mark("rotary")
+            if hw == self.value_dim:             # the heads' results are as wide as they have to be: gated in place
+                self._attend(qh, y, hw, k_packed=kh, v_packed=vh, n_kv_heads=H, gate=gate, **common)
+                kernels.mark("attention")
+            else:
+                oh = torch.empty((T, H * hw), dtype=act, device=dev)
+                self._attend(qh, oh, hw, k_packed=kh, v_packed=vh, n_kv_heads=H, **common)
+                kernels.mark("attention")
+                kernels.latent_expand(oh, None, y, heads=H, kv_rank=hw, row_width=hw, value_dim=self.value_dim, gate=gate,
+                                      head_gate=self.head_gate)
+                kernels.mark("rotary")
             kernels.linear(y, self.w_o, out=residual, accumulate=not ctx.store_result)
             kernels.mark("o")
             return
@@ -238,9 +251,10 @@ class LatentAttention(Mixer):
         kernels.linear(y, self.w_o, out=residual, accumulate=not ctx.store_result)
         kernels.mark("o")
 
-    def _attend(self, q, out, width, **kw):
-        """The attention kernels over rows of `width` entries, with the sink if there is one."""
-        if self.sinks is None:
+    def _attend(self, q, out, width, gate=None, **kw):
+        """The attention kernels over rows of `width` entries, with the sink and the gate if there are any."""
+        if self.sinks is None and gate is None:
             kernels.attention(q, out, head_dim=width, **kw)
         else:
-            kernels.attention_ext(q, out, key_dim=width, value_dim=width, sink=self.sinks, **kw)
+            kernels.attention_ext(q, out, key_dim=width, value_dim=width, gate=gate,
+                                  sink=False if self.sinks is None else self.sinks, **kw)
