@@ -265,7 +265,7 @@ template <typename TA, bool KN>
 __global__ void __launch_bounds__(128)
 latent_product_kernel(const TA* __restrict__ a, int lda, int a_head, const bf16* __restrict__ w, int H, int K, int N,
                       bf16* __restrict__ out, int out_head, int n_tokens, LpQuery qq, const float* __restrict__ gate,
-                      int ldg, int head_gate) {
+                      int ldg, int head_gate, int a_vec) {
     constexpr int AW = LP_KC + 8;                              // padded rows: ldmatrix without bank conflicts
     constexpr int BW = KN ? LP_COLS + 8 : LP_KC + 8;
     constexpr int BROWS = KN ? LP_KC : LP_COLS;
@@ -277,13 +277,19 @@ latent_product_kernel(const TA* __restrict__ a, int lda, int a_head, const bf16*
     const bf16* wh = w + (size_t)h * K * N;
     // the first piece of the head's matrix does not depend on the kernel before
     auto load_b = [&](int k0) {
-        for (int p = threadIdx.x; p < BROWS * (KN ? LP_COLS : LP_KC) / 8; p += 128) {
-            const int per = (KN ? LP_COLS : LP_KC) / 8;
-            const int row = p / per, c = (p - row * per) * 8;
+        constexpr int PER = (KN ? LP_COLS : LP_KC) / 8, COPIES = BROWS * PER / 128;
+        uint4 v[COPIES];                                       // all loads in flight before the first store
+#pragma unroll
+        for (int i = 0; i < COPIES; ++i) {
+            const int p = threadIdx.x + 128 * i, row = p / PER, c = (p - row * PER) * 8;
             const int k = KN ? k0 + row : k0 + c, n = KN ? c0 + c : c0 + row;
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (k < K && n < N) v = *reinterpret_cast<const uint4*>(wh + (KN ? (size_t)k * N + n : (size_t)n * K + k));
-            *reinterpret_cast<uint4*>(b_s + row * BW + c) = v;
+            v[i] = make_uint4(0u, 0u, 0u, 0u);
+            if (k < K && n < N) v[i] = *reinterpret_cast<const uint4*>(wh + (KN ? (size_t)k * N + n : (size_t)n * K + k));
+        }
+#pragma unroll
+        for (int i = 0; i < COPIES; ++i) {
+            const int p = threadIdx.x + 128 * i, row = p / PER, c = (p - row * PER) * 8;
+            *reinterpret_cast<uint4*>(b_s + row * BW + c) = v[i];
         }
     };
     load_b(0);
@@ -295,16 +301,40 @@ latent_product_kernel(const TA* __restrict__ a, int lda, int a_head, const bf16*
     for (int k0 = 0; k0 < K; k0 += LP_KC) {
         const int kc = min(LP_KC, (K - k0 + 15) & ~15);
         if (k0 > 0) { __syncthreads(); load_b(k0); }
-        for (int p = threadIdx.x; p < LP_TOK * LP_KC / 2; p += 128) {
-            const int row = p / (LP_KC / 2), c = (p - row * (LP_KC / 2)) * 2, t = t0 + row, k = k0 + c;
-            bf16 v0 = zero, v1 = zero;
-            if (t < n_tokens) {
-                const TA* ar = a + (size_t)t * lda + (size_t)h * a_head;
-                if (k < K) v0 = from_f32<bf16>(to_f32<TA>(ar[k]));
-                if (k + 1 < K) v1 = from_f32<bf16>(to_f32<TA>(ar[k + 1]));
+        if (a_vec) {                                           // rows of whole 16-byte pieces: four entries at a time
+            constexpr int COPIES = LP_TOK * LP_KC / 4 / 128;
+            float v[COPIES][4];
+#pragma unroll
+            for (int i = 0; i < COPIES; ++i) {
+                const int p = threadIdx.x + 128 * i, row = p / (LP_KC / 4), k = k0 + (p - row * (LP_KC / 4)) * 4;
+                v[i][0] = v[i][1] = v[i][2] = v[i][3] = 0.f;
+                if (t0 + row < n_tokens && k < K) {
+                    const TA* ar = a + (size_t)(t0 + row) * lda + (size_t)h * a_head + k;
+                    if constexpr (sizeof(TA) == 4) load16_f32<TA>(ar, v[i]);
+                    else {
+                        const float2 x = load2_f32<TA>(ar), y = load2_f32<TA>(ar + 2);
+                        v[i][0] = x.x; v[i][1] = x.y; v[i][2] = y.x; v[i][3] = y.y;
+                    }
+                }
             }
-            a_s[row * AW + c] = v0;
-            a_s[row * AW + c + 1] = v1;
+#pragma unroll
+            for (int i = 0; i < COPIES; ++i) {
+                const int p = threadIdx.x + 128 * i, row = p / (LP_KC / 4), c = (p - row * (LP_KC / 4)) * 4;
+                store2_f32<bf16>(a_s + row * AW + c, v[i][0], v[i][1]);
+                store2_f32<bf16>(a_s + row * AW + c + 2, v[i][2], v[i][3]);
+            }
+        } else {
+            for (int p = threadIdx.x; p < LP_TOK * LP_KC / 2; p += 128) {
+                const int row = p / (LP_KC / 2), c = (p - row * (LP_KC / 2)) * 2, t = t0 + row, k = k0 + c;
+                bf16 v0 = zero, v1 = zero;
+                if (t < n_tokens) {
+                    const TA* ar = a + (size_t)t * lda + (size_t)h * a_head;
+                    if (k < K) v0 = from_f32<bf16>(to_f32<TA>(ar[k]));
+                    if (k + 1 < K) v1 = from_f32<bf16>(to_f32<TA>(ar[k + 1]));
+                }
+                a_s[row * AW + c] = v0;
+                a_s[row * AW + c + 1] = v1;
+            }
         }
         __syncthreads();
         const int mat = lane >> 3, r8 = lane & 7;
@@ -382,7 +412,8 @@ TQ_API int tq_latent_query(const float* q, int ldq, int H, int d, int r, int n, 
         return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_product_kernel<float, true>,
                              dim3(H, (n + LP_COLS - 1) / LP_COLS, (n_tokens + LP_TOK - 1) / LP_TOK), dim3(128), 0, stream, q,
                              ldq, d + r, (const bf16*)uk, H, d, n, (bf16*)out, rp, n_tokens,
-                             LpQuery{d, r, rp, rot_dims, paired, cos_t, sin_t, tok_pos}, (const float*)nullptr, 0, 0);
+                             LpQuery{d, r, rp, rot_dims, paired, cos_t, sin_t, tok_pos}, (const float*)nullptr, 0, 0,
+                             (int)(!((ldq | d | r) & 3) && (reinterpret_cast<uintptr_t>(q) & 15) == 0));
     const int threads = rp > 128 ? 256 : 128;
     const size_t smem = (size_t)(d + r) * sizeof(float);
     const dim3 grid(n_tokens, H);
@@ -404,7 +435,8 @@ TQ_API int tq_latent_expand(const void* lat, int H, int n, int rp, int e, const 
         return tq_launch_pdl(TQ_PDL_ELEMENTWISE, latent_product_kernel<bf16, false>,
                              dim3(H, (e + LP_COLS - 1) / LP_COLS, (n_tokens + LP_TOK - 1) / LP_TOK), dim3(128), 0, stream,
                              (const bf16*)lat, H * rp, rp, (const bf16*)uv, H, n, e, (bf16*)out, e, n_tokens,
-                             LpQuery{0, 0, 0, 0, 0, nullptr, nullptr, nullptr}, gate, ldg, head_gate);
+                             LpQuery{0, 0, 0, 0, 0, nullptr, nullptr, nullptr}, gate, ldg, head_gate,
+                             (int)(!((rp | n) & 3) && (reinterpret_cast<uintptr_t>(lat) & 7) == 0));
     const size_t smem = (size_t)n * sizeof(float);
     const dim3 grid(n_tokens, H);
     if (dtype == TQ_F32)

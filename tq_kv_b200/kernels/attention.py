@@ -24,6 +24,11 @@ def check_head_geometry(n_heads: int, n_kv_heads: int, head_dim: int) -> None:
         raise KernelError(f"attention: more than 65535 key/value heads ({n_kv_heads})")
 
 
+def head_groups(n_heads: int, n_kv_heads: int) -> int:
+    """Blocks per token of the decode kernel: it serves up to 16 query heads of a key/value head at once."""
+    return n_kv_heads * -(-(n_heads // n_kv_heads) // 16)
+
+
 def plan_splits(n_tokens: int, n_kv_heads: int, max_keys: int, sm_count: int) -> int:
     """Number of splits of the key range for a step: one while the grid fills
     the GPU or the key ranges are short, else as many as fill the GPU in one

@@ -237,7 +237,7 @@ class LatentAttention(Mixer):
         kernels.mark("rotary")
         lat = torch.empty_like(qa)
         max_keys = b.max_new_len if self.window is None else min(b.max_new_len, self.window)
-        n_splits = kernels.plan_splits(T, 1, max_keys, ctx.runtime.sm_count)
+        n_splits = kernels.plan_splits(T, kernels.head_groups(H, 1), max_keys, ctx.runtime.sm_count)
         scratch = None
         if n_splits > 1:
             scratch = torch.empty(kernels.split_scratch_floats(T, H, row, n_splits), dtype=torch.float32, device=dev)

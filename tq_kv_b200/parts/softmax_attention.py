@@ -340,7 +340,7 @@ class SoftmaxAttention(Mixer):
             parts = kernels.attention_ext(q, into, k_packed=k, v_packed=v, **common)
         else:
             max_keys = b.max_new_len if self.span is None else min(b.max_new_len, self.span + self.keep_first)
-            n_splits = kernels.plan_splits(T, self.n_kv_heads, max_keys, ctx.runtime.sm_count)
+            n_splits = kernels.plan_splits(T, kernels.head_groups(self.n_heads * self.maps, self.n_kv_heads), max_keys, ctx.runtime.sm_count)
             scratch = None
             if n_splits > 1:
                 scratch = torch.empty(kernels.split_scratch_floats(T, self.n_heads * self.maps, self.value_row, n_splits),
