@@ -136,6 +136,116 @@ head_encode_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col,
     }
 }
 
+// The same for vectors of up to 128 entries in pieces of four (hd, rot / 2, vd, kr, vr, the columns and the row stride
+// multiples of four, halves layout, values of their own, no whole-row norm): LPV lanes per vector, four neighbouring
+// entries per lane, the partner entries of a rotation by shuffles, 8-byte (16-byte) stores.
+template <typename TC> __device__ __forceinline__ void he_store4(TC* p, const float* v);
+template <> __device__ __forceinline__ void he_store4<float>(float* p, const float* v) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+template <> __device__ __forceinline__ void he_store4<bf16>(bf16* p, const float* v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+template <typename TC, int LPV>
+__global__ void __launch_bounds__(128)
+head_encode4_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, int v_col,
+                    const float* __restrict__ cos_tab, const float* __restrict__ sin_tab, int rot, float norm_eps,
+                    const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ new_lens,
+                    const int* __restrict__ block_table, int table_width, int ring_pages, int page_tokens,
+                    TC* __restrict__ q_out, TC* __restrict__ k_out, TC* __restrict__ v_out, TC* __restrict__ k_pages,
+                    TC* __restrict__ v_pages, int nh, int nkv, int hd, int vd, const float* __restrict__ q_w,
+                    const float* __restrict__ k_w, float v_scale, int maps, int kr, int vr) {
+    constexpr int PER_WARP = 32 / LPV;
+    const int t = blockIdx.x, lane = threadIdx.x & 31, part = lane & (LPV - 1);
+    const int nq = nh * maps, nk = nkv * maps;
+    const int head = (blockIdx.y * 4 + (threadIdx.x >> 5)) * PER_WARP + lane / LPV;
+    const bool live = head < nq + nk + nkv;                    // (dead lanes stay for the shuffles)
+    const int pos = tok_pos[t];
+    const int b = tok_seq[t];
+    const bool is_q = head < nq, is_k = !is_q && head < nq + nk;
+    const int g = is_q ? head : (is_k ? head - nq : head - nq - nk);
+    const int map = g % maps, map_off = is_q || is_k ? map * hd : 0;
+    const int width = (is_q || is_k) ? hd : vd, row_w = (is_q || is_k) ? kr : vr;
+    const int d0 = part * 4;
+    const bool mine = live && d0 < width;
+    TC *dst = nullptr, *cache = nullptr;
+    if (live) {
+        const int kvh = is_k ? g / maps : g;
+        if (is_q) dst = q_out + ((size_t)t * nq + g) * kr;
+        else if (is_k) dst = k_out ? k_out + ((size_t)t * nkv + kvh) * kr : nullptr;
+        else dst = v_out ? v_out + ((size_t)t * nkv + kvh) * vr : nullptr;
+        if (!is_q && k_pages != nullptr) {
+            int lp = pos / page_tokens;
+            bool keep = pos < new_lens[b];
+            if (ring_pages > 0) {
+                keep = keep && pos >= new_lens[b] - ring_pages * page_tokens;
+                lp %= ring_pages;
+            }
+            if (keep) {
+                const int page = block_table[(size_t)b * table_width + lp];
+                const size_t row = ((size_t)page * nkv + kvh) * page_tokens + (pos % page_tokens);
+                cache = is_k ? k_pages + row * kr : v_pages + row * vr;
+            }
+        }
+    }
+    const int half = rot >> 1;
+    float w[4] = {1.f, 1.f, 1.f, 1.f}, cs[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
+    const bool turns = mine && (is_q || is_k) && d0 < rot;
+    if (mine && (is_q || is_k)) {                              // weights and tables do not depend on the kernel before
+        const float* ww = is_q ? q_w : k_w;
+        if (ww) load16_f32<float>(ww + d0, w);
+        if (turns) {
+            const int j = d0 < half ? d0 : d0 - half;
+            load16_f32<float>(cos_tab + (size_t)pos * half + j, cs);
+            load16_f32<float>(sin_tab + (size_t)pos * half + j, sn);
+        }
+    }
+    pdl_wait();
+    pdl_launch();
+    float x[4] = {0.f, 0.f, 0.f, 0.f};
+    if (mine)
+        load16_f32<float>(proj + (size_t)t * ld + (is_q ? q_col + g * hd : (is_k ? k_col + g * hd : v_col + g * vd)) + d0, x);
+    float inv = 1.f;
+    if (norm_eps > 0.f) {
+        float ss = fmaf(x[0], x[0], fmaf(x[1], x[1], fmaf(x[2], x[2], x[3] * x[3])));
+#pragma unroll
+        for (int o = LPV / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        inv = 1.f / sqrtf(ss / (float)width + norm_eps);
+    }
+    if (is_q || is_k) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[e] = x[e] * inv * w[e];
+    } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[e] *= v_scale;
+    }
+    if (half > 0) {                                            // entry i < half pairs with entry i + half, half / 4 lanes on
+        const int step = half >> 2;
+        const bool low = d0 < half;
+        const int from = (lane & ~(LPV - 1)) + ((low ? part + step : part - step) & (LPV - 1));
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float y = __shfl_sync(0xffffffffu, x[e], from);
+            if (turns) x[e] = low ? x[e] * cs[e] - y * sn[e] : x[e] * cs[e] + y * sn[e];
+        }
+    }
+    if (mine) {
+        if (dst) he_store4<TC>(dst + map_off + d0, x);
+        if (cache) he_store4<TC>(cache + map_off + d0, x);
+    }
+    if (!live) return;
+    // zeros: around a map's query; behind a key row's last map; behind a value row
+    const float none[4] = {0.f, 0.f, 0.f, 0.f};
+    const int z0 = is_q ? 0 : (is_k ? (map == maps - 1 ? maps * hd : row_w) : vd);
+    for (int d = z0 + d0; d < row_w; d += 4 * LPV) {
+        if (is_q && d >= map_off && d < map_off + hd) continue;
+        if (dst) he_store4<TC>(dst + d, none);
+        if (cache) he_store4<TC>(cache + d, none);
+    }
+}
+
 TQ_API int tq_head_encode(const float* proj, int ld, int q_col, int k_col, int v_col, const float* cos_tab,
                           const float* sin_tab, int rot, float norm_eps, const int* tok_pos, const int* tok_seq,
                           const int* new_lens, const int* block_table, int table_width, int ring_pages,
@@ -153,7 +263,34 @@ TQ_API int tq_head_encode(const float* proj, int ld, int q_col, int k_col, int v
     if ((k_pages == nullptr) != (v_pages == nullptr)) return (int)cudaErrorInvalidValue;
     if (k_pages && !block_table) return (int)cudaErrorInvalidValue;
     if (nkv > 0 && v_col < 0 && vd != hd) return (int)cudaErrorInvalidValue;
-    const int groups = (nh * maps + nkv * maps + nkv + 3) / 4;
+    const int vectors = nh * maps + nkv * maps + nkv;
+    const int widest = hd > vd ? hd : vd;
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    if (!row_inv && !paired && v_col >= 0 && widest <= 128 && !((hd | (rot >> 1) | vd | kr | vr | ld | q_col | k_col | v_col) & 3) &&
+        aligned(proj) && aligned(q_out) && aligned(k_out) && aligned(v_out) && aligned(k_pages) && aligned(v_pages) &&
+        aligned(cos_tab) && aligned(sin_tab) && aligned(q_w) && aligned(k_w)) {
+        const int lpv = widest <= 32 ? 8 : (widest <= 64 ? 16 : 32), per_block = 4 * (32 / lpv);
+        const int blocks = (vectors + per_block - 1) / per_block;
+        if (blocks > 65535) return (int)cudaErrorInvalidValue;
+#define TQ_LAUNCH4(TC, L)                                                                                               \
+    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, head_encode4_kernel<TC, L>, dim3(n_tokens, blocks), dim3(128), 0, stream,   \
+                         proj, ld, q_col, k_col, v_col, cos_tab, sin_tab, rot, norm_eps, tok_pos, tok_seq, new_lens,     \
+                         block_table, table_width, ring_pages, page_tokens, (TC*)q_out, (TC*)k_out, (TC*)v_out,          \
+                         (TC*)k_pages, (TC*)v_pages, nh, nkv, hd, vd, q_w, k_w, v_scale, maps, kr, vr)
+        if (cache_dtype == TQ_F32) {
+            if (lpv == 8) TQ_LAUNCH4(float, 8);
+            if (lpv == 16) TQ_LAUNCH4(float, 16);
+            TQ_LAUNCH4(float, 32);
+        }
+        if (cache_dtype == TQ_BF16) {
+            if (lpv == 8) TQ_LAUNCH4(bf16, 8);
+            if (lpv == 16) TQ_LAUNCH4(bf16, 16);
+            TQ_LAUNCH4(bf16, 32);
+        }
+#undef TQ_LAUNCH4
+        return (int)cudaErrorInvalidValue;
+    }
+    const int groups = (vectors + 3) / 4;
     if (groups > 65535) return (int)cudaErrorInvalidValue;
     const dim3 grid(n_tokens, groups);
 #define TQ_LAUNCH(TC)                                                                                              \
@@ -206,8 +343,8 @@ TQ_API int tq_row_inv_rms(const float* proj, int ld, int q_col, int q_n, int q_c
 // unnormalised sums over n_splits shares of the keys with their maxima and sums of weights (natural-log units), which
 // are merged here in index order, as attention_merge_kernel does.  A warp per (token, head).
 // ---------------------------------------------------------------------------
-#define DM_MAX_PER_LANE 16    // e <= 512
-template <typename TO>
+// V: entries a lane takes at a time (4: rows and heads of whole 16-byte pieces; 1: any), PER: how often.
+template <typename TO, int V, int PER>
 __global__ void __launch_bounds__(128)
 difference_of_maps_kernel(const float* __restrict__ a, const float* __restrict__ ml, int n_splits, int row, int e, int H,
                           float factor, float eps, float out_scale, const float* __restrict__ gate, int ldg,
@@ -217,16 +354,32 @@ difference_of_maps_kernel(const float* __restrict__ a, const float* __restrict__
     const int t = pair / H, h = pair - t * H;
     pdl_wait();
     pdl_launch();
-    float o[DM_MAX_PER_LANE];
+    float o[PER][V];
 #pragma unroll
-    for (int i = 0; i < DM_MAX_PER_LANE; ++i) o[i] = 0.f;
+    for (int i = 0; i < PER; ++i)
+#pragma unroll
+        for (int c = 0; c < V; ++c) o[i][c] = 0.f;
+    auto add = [&](const float* src, float f) {                        // o += f * src
+        float v[PER][V];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int d = V * (lane + 32 * i);
+#pragma unroll
+            for (int c = 0; c < V; ++c) v[i][c] = 0.f;
+            if (d < e) {
+                if constexpr (V == 4) load16_f32<float>(src + d, v[i]);
+                else v[i][0] = src[d];
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+#pragma unroll
+            for (int c = 0; c < V; ++c) o[i][c] = fmaf(f, v[i][c], o[i][c]);
+    };
     const float* r0 = a + (size_t)pair * 2 * n_splits * row;           // [2 maps][n_splits][row]
     if (!ml) {
-#pragma unroll
-        for (int i = 0; i < DM_MAX_PER_LANE; ++i) {
-            const int d = lane + 32 * i;
-            if (d < e) o[i] = fmaf(-factor, r0[row + d], r0[d]);
-        }
+        add(r0, 1.f);
+        add(r0 + row, -factor);
     } else {
         for (int m = 0; m < 2; ++m) {
             const float* mls = ml + ((size_t)pair * 2 + m) * n_splits * 2;
@@ -241,28 +394,27 @@ difference_of_maps_kernel(const float* __restrict__ a, const float* __restrict__
             const float sign = (m ? -factor : 1.f) / l;
             for (int s = 0; s < n_splits; ++s) {
                 const float ms = mls[2 * s];
-                const float f = ms > -INFINITY ? expf(ms - mx) * sign : 0.f;
-#pragma unroll
-                for (int i = 0; i < DM_MAX_PER_LANE; ++i) {
-                    const int d = lane + 32 * i;
-                    if (d < e) {
-                        const float v = acc[(size_t)s * row + d];
-                        o[i] += ms > -INFINITY ? v * f : 0.f;         // (an empty share's sums are not looked at)
-                    }
-                }
+                if (ms > -INFINITY) add(acc + (size_t)s * row, expf(ms - mx) * sign);    // (an empty share holds nothing)
             }
         }
     }
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < DM_MAX_PER_LANE; ++i) ss = fmaf(o[i], o[i], ss);
+    for (int i = 0; i < PER; ++i)
+#pragma unroll
+        for (int c = 0; c < V; ++c) ss = fmaf(o[i][c], o[i][c], ss);
     ss = warp_sum(ss);
     float f = out_scale / sqrtf(ss / (float)e + eps);
     if (gate) f *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + h]));
 #pragma unroll
-    for (int i = 0; i < DM_MAX_PER_LANE; ++i) {
-        const int d = lane + 32 * i;
-        if (d < e) out[(size_t)pair * e + d] = from_f32<TO>(o[i] * f);
+    for (int i = 0; i < PER; ++i) {
+        const int d = V * (lane + 32 * i);
+        if (d < e) {
+#pragma unroll
+            for (int c = 0; c < V; ++c) o[i][c] *= f;
+            if constexpr (V == 4) he_store4<TO>(out + (size_t)pair * e + d, o[i]);
+            else out[(size_t)pair * e + d] = from_f32<TO>(o[i][0]);
+        }
     }
 }
 
@@ -270,17 +422,25 @@ TQ_API int tq_difference_of_maps(const float* a, const float* ml, int n_splits, 
                                  float eps, float out_scale, const float* gate, int ldg, void* out, int dtype,
                                  int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (!a || !out || n_splits < 1 || (!ml && n_splits != 1) || e <= 0 || e > 32 * DM_MAX_PER_LANE || row < e || heads <= 0)
+    if (!a || !out || n_splits < 1 || (!ml && n_splits != 1) || e <= 0 || e > 512 || row < e || heads <= 0)
         return (int)cudaErrorInvalidValue;
     if ((long long)n_tokens * heads > 0x7fffffffll - 4) return (int)cudaErrorInvalidValue;
     const int n_pairs = n_tokens * heads;
     const dim3 grid((n_pairs + 3) / 4);
-    if (dtype == TQ_F32)
-        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, difference_of_maps_kernel<float>, grid, dim3(128), 0, stream, a, ml, n_splits,
-                             row, e, heads, factor, eps, out_scale, gate, ldg, (float*)out, n_pairs);
-    if (dtype == TQ_BF16)
-        return tq_launch_pdl(TQ_PDL_ELEMENTWISE, difference_of_maps_kernel<bf16>, grid, dim3(128), 0, stream, a, ml, n_splits,
-                             row, e, heads, factor, eps, out_scale, gate, ldg, (bf16*)out, n_pairs);
+    const bool vec = !((e | row) & 3) && ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+#define TQ_DM(TO, V, PER)                                                                                               \
+    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, difference_of_maps_kernel<TO, V, PER>, grid, dim3(128), 0, stream, a, ml,    \
+                         n_splits, row, e, heads, factor, eps, out_scale, gate, ldg, (TO*)out, n_pairs)
+#define TQ_DM_SIZES(TO)                                                                                                 \
+    do {                                                                                                                \
+        if (vec && e <= 128) TQ_DM(TO, 4, 1);                                                                           \
+        if (vec) TQ_DM(TO, 4, 4);                                                                                       \
+        TQ_DM(TO, 1, 16);                                                                                               \
+    } while (0)
+    if (dtype == TQ_F32) TQ_DM_SIZES(float);
+    if (dtype == TQ_BF16) TQ_DM_SIZES(bf16);
+#undef TQ_DM_SIZES
+#undef TQ_DM
     return (int)cudaErrorInvalidValue;
 }
 
