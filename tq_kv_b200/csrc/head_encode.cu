@@ -136,9 +136,10 @@ head_encode_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col,
     }
 }
 
-// The same for vectors of up to 128 entries in pieces of four (hd, rot / 2, vd, kr, vr, the columns and the row stride
-// multiples of four, halves layout, values of their own, no whole-row norm): LPV lanes per vector, four neighbouring
-// entries per lane, the partner entries of a rotation by shuffles, 8-byte (16-byte) stores.
+// The same for heads of up to 128 entries in pieces of four (hd, rot / 2, vd, kr, vr, the columns and the row stride
+// multiples of four, halves layout, values of their own, no whole-row norm, one or two maps): LPV lanes per head, four
+// neighbouring entries per lane, a head's maps one after the other with the same weights and table entries, the
+// partner entries of a rotation by shuffles, 8-byte (16-byte) stores.
 template <typename TC> __device__ __forceinline__ void he_store4(TC* p, const float* v);
 template <> __device__ __forceinline__ void he_store4<float>(float* p, const float* v) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
@@ -148,7 +149,7 @@ template <> __device__ __forceinline__ void he_store4<bf16>(bf16* p, const float
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
 }
 
-template <typename TC, int LPV>
+template <typename TC, int LPV, int MAPS>
 __global__ void __launch_bounds__(128)
 head_encode4_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, int v_col,
                     const float* __restrict__ cos_tab, const float* __restrict__ sin_tab, int rot, float norm_eps,
@@ -156,93 +157,105 @@ head_encode4_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col
                     const int* __restrict__ block_table, int table_width, int ring_pages, int page_tokens,
                     TC* __restrict__ q_out, TC* __restrict__ k_out, TC* __restrict__ v_out, TC* __restrict__ k_pages,
                     TC* __restrict__ v_pages, int nh, int nkv, int hd, int vd, const float* __restrict__ q_w,
-                    const float* __restrict__ k_w, float v_scale, int maps, int kr, int vr) {
+                    const float* __restrict__ k_w, float v_scale, int kr, int vr) {
     constexpr int PER_WARP = 32 / LPV;
-    const int t = blockIdx.x, lane = threadIdx.x & 31, part = lane & (LPV - 1);
-    const int nq = nh * maps, nk = nkv * maps;
+    const int t = blockIdx.x, lane = threadIdx.x & 31, part = lane & (LPV - 1), d0 = part * 4;
     const int head = (blockIdx.y * 4 + (threadIdx.x >> 5)) * PER_WARP + lane / LPV;
-    const bool live = head < nq + nk + nkv;                    // (dead lanes stay for the shuffles)
+    const bool live = head < nh + 2 * nkv;                     // (dead lanes stay for the shuffles)
+    const bool is_q = head < nh, is_k = !is_q && head < nh + nkv;
+    const int g = is_q ? head : (is_k ? head - nh : head - nh - nkv);
     const int pos = tok_pos[t];
-    const int b = tok_seq[t];
-    const bool is_q = head < nq, is_k = !is_q && head < nq + nk;
-    const int g = is_q ? head : (is_k ? head - nq : head - nq - nk);
-    const int map = g % maps, map_off = is_q || is_k ? map * hd : 0;
-    const int width = (is_q || is_k) ? hd : vd, row_w = (is_q || is_k) ? kr : vr;
-    const int d0 = part * 4;
-    const bool mine = live && d0 < width;
-    TC *dst = nullptr, *cache = nullptr;
+    TC *dst = nullptr, *cache = nullptr;                       // this head's row(s), and its row in the cache
     if (live) {
-        const int kvh = is_k ? g / maps : g;
-        if (is_q) dst = q_out + ((size_t)t * nq + g) * kr;
-        else if (is_k) dst = k_out ? k_out + ((size_t)t * nkv + kvh) * kr : nullptr;
-        else dst = v_out ? v_out + ((size_t)t * nkv + kvh) * vr : nullptr;
+        if (is_q) dst = q_out + ((size_t)t * nh + g) * MAPS * kr;
+        else if (is_k) dst = k_out ? k_out + ((size_t)t * nkv + g) * kr : nullptr;
+        else dst = v_out ? v_out + ((size_t)t * nkv + g) * vr : nullptr;
         if (!is_q && k_pages != nullptr) {
+            const int b = tok_seq[t], n = new_lens[b];
             int lp = pos / page_tokens;
-            bool keep = pos < new_lens[b];
+            const int in_page = pos - lp * page_tokens;
+            bool keep = pos < n;
             if (ring_pages > 0) {
-                keep = keep && pos >= new_lens[b] - ring_pages * page_tokens;
+                keep = keep && pos >= n - ring_pages * page_tokens;
                 lp %= ring_pages;
             }
             if (keep) {
-                const int page = block_table[(size_t)b * table_width + lp];
-                const size_t row = ((size_t)page * nkv + kvh) * page_tokens + (pos % page_tokens);
+                const size_t row = ((size_t)block_table[(size_t)b * table_width + lp] * nkv + g) * page_tokens + in_page;
                 cache = is_k ? k_pages + row * kr : v_pages + row * vr;
             }
         }
     }
     const int half = rot >> 1;
+    const bool mine = live && (is_q || is_k) && d0 < hd, turns = mine && d0 < rot, low = d0 < half;
     float w[4] = {1.f, 1.f, 1.f, 1.f}, cs[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
-    const bool turns = mine && (is_q || is_k) && d0 < rot;
-    if (mine && (is_q || is_k)) {                              // weights and tables do not depend on the kernel before
+    if (mine) {                                                // weights and tables do not depend on the kernel before
         const float* ww = is_q ? q_w : k_w;
         if (ww) load16_f32<float>(ww + d0, w);
         if (turns) {
-            const int j = d0 < half ? d0 : d0 - half;
+            const int j = low ? d0 : d0 - half;
             load16_f32<float>(cos_tab + (size_t)pos * half + j, cs);
             load16_f32<float>(sin_tab + (size_t)pos * half + j, sn);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sn[e] = low ? -sn[e] : sn[e];
         }
     }
     pdl_wait();
     pdl_launch();
-    float x[4] = {0.f, 0.f, 0.f, 0.f};
-    if (mine)
-        load16_f32<float>(proj + (size_t)t * ld + (is_q ? q_col + g * hd : (is_k ? k_col + g * hd : v_col + g * vd)) + d0, x);
-    float inv = 1.f;
-    if (norm_eps > 0.f) {
-        float ss = fmaf(x[0], x[0], fmaf(x[1], x[1], fmaf(x[2], x[2], x[3] * x[3])));
+    const float* src = proj + (size_t)t * ld;
+    const float none[4] = {0.f, 0.f, 0.f, 0.f};
+    if (live && !is_q && !is_k) {                              // values: copied, zeros behind
+        for (int d = d0; d < vr; d += 4 * LPV) {
+            float x[4] = {0.f, 0.f, 0.f, 0.f};
+            if (d < vd) load16_f32<float>(src + v_col + g * vd + d, x);
 #pragma unroll
-        for (int o = LPV / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        inv = 1.f / sqrtf(ss / (float)width + norm_eps);
-    }
-    if (is_q || is_k) {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) x[e] = x[e] * inv * w[e];
-    } else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) x[e] *= v_scale;
-    }
-    if (half > 0) {                                            // entry i < half pairs with entry i + half, half / 4 lanes on
-        const int step = half >> 2;
-        const bool low = d0 < half;
-        const int from = (lane & ~(LPV - 1)) + ((low ? part + step : part - step) & (LPV - 1));
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const float y = __shfl_sync(0xffffffffu, x[e], from);
-            if (turns) x[e] = low ? x[e] * cs[e] - y * sn[e] : x[e] * cs[e] + y * sn[e];
+            for (int e = 0; e < 4; ++e) x[e] *= v_scale;
+            if (dst) he_store4<TC>(dst + d, x);
+            if (cache) he_store4<TC>(cache + d, x);
         }
     }
-    if (mine) {
-        if (dst) he_store4<TC>(dst + map_off + d0, x);
-        if (cache) he_store4<TC>(cache + map_off + d0, x);
+    float x[MAPS][4];
+#pragma unroll
+    for (int m = 0; m < MAPS; ++m) {
+        x[m][0] = x[m][1] = x[m][2] = x[m][3] = 0.f;
+        if (mine) load16_f32<float>(src + (is_q ? q_col : k_col) + (g * MAPS + m) * hd + d0, x[m]);
     }
-    if (!live) return;
-    // zeros: around a map's query; behind a key row's last map; behind a value row
-    const float none[4] = {0.f, 0.f, 0.f, 0.f};
-    const int z0 = is_q ? 0 : (is_k ? (map == maps - 1 ? maps * hd : row_w) : vd);
-    for (int d = z0 + d0; d < row_w; d += 4 * LPV) {
-        if (is_q && d >= map_off && d < map_off + hd) continue;
-        if (dst) he_store4<TC>(dst + d, none);
-        if (cache) he_store4<TC>(cache + d, none);
+    // entry i < half pairs with entry i + half, half / 4 lanes on
+    const int from = (lane & ~(LPV - 1)) + ((low ? part + (half >> 2) : part - (half >> 2)) & (LPV - 1));
+#pragma unroll
+    for (int m = 0; m < MAPS; ++m) {
+        float inv = 1.f;
+        if (norm_eps > 0.f) {
+            float ss = fmaf(x[m][0], x[m][0], fmaf(x[m][1], x[m][1], fmaf(x[m][2], x[m][2], x[m][3] * x[m][3])));
+#pragma unroll
+            for (int o = LPV / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            inv = 1.f / sqrtf(ss / (float)hd + norm_eps);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[m][e] = x[m][e] * inv * w[e];
+        if (half > 0) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float y = __shfl_sync(0xffffffffu, x[m][e], from);
+                if (turns) x[m][e] = x[m][e] * cs[e] + y * sn[e];
+            }
+        }
+        if (mine) {
+            if (dst) he_store4<TC>(dst + (is_q ? m * kr : 0) + m * hd + d0, x[m]);
+            if (cache) he_store4<TC>(cache + m * hd + d0, x[m]);
+        }
+    }
+    if (!live || !(is_q || is_k)) return;
+    // zeros: around each map's query, behind a key row's last map
+    if (is_q) {
+#pragma unroll
+        for (int m = 0; m < MAPS; ++m)
+            for (int d = d0; d < kr; d += 4 * LPV)
+                if (d < m * hd || d >= m * hd + hd) he_store4<TC>(dst + m * kr + d, none);
+    } else {
+        for (int d = MAPS * hd + d0; d < kr; d += 4 * LPV) {
+            if (dst) he_store4<TC>(dst + d, none);
+            if (cache) he_store4<TC>(cache + d, none);
+        }
     }
 }
 
@@ -264,29 +277,30 @@ TQ_API int tq_head_encode(const float* proj, int ld, int q_col, int k_col, int v
     if (k_pages && !block_table) return (int)cudaErrorInvalidValue;
     if (nkv > 0 && v_col < 0 && vd != hd) return (int)cudaErrorInvalidValue;
     const int vectors = nh * maps + nkv * maps + nkv;
-    const int widest = hd > vd ? hd : vd;
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    if (!row_inv && !paired && v_col >= 0 && widest <= 128 && !((hd | (rot >> 1) | vd | kr | vr | ld | q_col | k_col | v_col) & 3) &&
-        aligned(proj) && aligned(q_out) && aligned(k_out) && aligned(v_out) && aligned(k_pages) && aligned(v_pages) &&
-        aligned(cos_tab) && aligned(sin_tab) && aligned(q_w) && aligned(k_w)) {
-        const int lpv = widest <= 32 ? 8 : (widest <= 64 ? 16 : 32), per_block = 4 * (32 / lpv);
-        const int blocks = (vectors + per_block - 1) / per_block;
+    if (!row_inv && !paired && v_col >= 0 && maps <= 2 && hd <= 128 &&
+        !((hd | (rot >> 1) | vd | kr | vr | ld | q_col | k_col | v_col) & 3) && aligned(proj) && aligned(q_out) &&
+        aligned(k_out) && aligned(v_out) && aligned(k_pages) && aligned(v_pages) && aligned(cos_tab) && aligned(sin_tab) &&
+        aligned(q_w) && aligned(k_w)) {
+        const int lpv = hd <= 32 ? 8 : (hd <= 64 ? 16 : 32), per_block = 4 * (32 / lpv);
+        const int blocks = (nh + 2 * nkv + per_block - 1) / per_block;
         if (blocks > 65535) return (int)cudaErrorInvalidValue;
-#define TQ_LAUNCH4(TC, L)                                                                                               \
-    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, head_encode4_kernel<TC, L>, dim3(n_tokens, blocks), dim3(128), 0, stream,   \
+#define TQ_LAUNCH4(TC, L, M)                                                                                            \
+    return tq_launch_pdl(TQ_PDL_ELEMENTWISE, head_encode4_kernel<TC, L, M>, dim3(n_tokens, blocks), dim3(128), 0, stream, \
                          proj, ld, q_col, k_col, v_col, cos_tab, sin_tab, rot, norm_eps, tok_pos, tok_seq, new_lens,     \
                          block_table, table_width, ring_pages, page_tokens, (TC*)q_out, (TC*)k_out, (TC*)v_out,          \
-                         (TC*)k_pages, (TC*)v_pages, nh, nkv, hd, vd, q_w, k_w, v_scale, maps, kr, vr)
-        if (cache_dtype == TQ_F32) {
-            if (lpv == 8) TQ_LAUNCH4(float, 8);
-            if (lpv == 16) TQ_LAUNCH4(float, 16);
-            TQ_LAUNCH4(float, 32);
-        }
-        if (cache_dtype == TQ_BF16) {
-            if (lpv == 8) TQ_LAUNCH4(bf16, 8);
-            if (lpv == 16) TQ_LAUNCH4(bf16, 16);
-            TQ_LAUNCH4(bf16, 32);
-        }
+                         (TC*)k_pages, (TC*)v_pages, nh, nkv, hd, vd, q_w, k_w, v_scale, kr, vr)
+#define TQ_LAUNCH4_SIZES(TC, M)                                                                                         \
+    do {                                                                                                                \
+        if (lpv == 8) TQ_LAUNCH4(TC, 8, M);                                                                             \
+        if (lpv == 16) TQ_LAUNCH4(TC, 16, M);                                                                           \
+        TQ_LAUNCH4(TC, 32, M);                                                                                          \
+    } while (0)
+        if (cache_dtype == TQ_F32 && maps == 1) TQ_LAUNCH4_SIZES(float, 1);
+        if (cache_dtype == TQ_F32) TQ_LAUNCH4_SIZES(float, 2);
+        if (cache_dtype == TQ_BF16 && maps == 1) TQ_LAUNCH4_SIZES(bf16, 1);
+        if (cache_dtype == TQ_BF16) TQ_LAUNCH4_SIZES(bf16, 2);
+#undef TQ_LAUNCH4_SIZES
 #undef TQ_LAUNCH4
         return (int)cudaErrorInvalidValue;
     }
