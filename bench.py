@@ -390,14 +390,14 @@ def safurax_config(width: int, ff: int, layers: int, vocab: int) -> dict:
     heads, kv = width // 128, max(1, width // 512)
     moe = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 2},
            "router": {"experts": SAFURAX_EXPERTS, "top": SAFURAX_TOP}}
-    maps = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5,
-            "rot": {"base": 1e4, "dims": 64, "scaling": {"factor": 4.0}}}
+    maps = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.4,
+            "rot": {"base": 5e4, "dims": 64, "scaling": {"factor": 8.0}}}
     plain = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 128, "q_rank": width // 2, "scale": 128 ** -0.5}
     windowed = {"heads": heads, "dim": 96, "rot_dim": 32, "vdim": 128, "kv_rank": 96, "scale": 128 ** -0.5,
                 "mask": {"size": SAFURAX_WINDOW}, "rot": {"base": 1e4, "dims": 32}}
     order = [("attention", maps, {"kind": "dense", "ff": ff}), ("latent_attention", plain, moe),
              ("latent_attention_2", windowed, moe), ("latent_attention_2", {**windowed, "kv_from": 2}, moe)]
-    return {"architecture": "Safurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 3.0},
+    return {"architecture": "Safurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 4.0},
             "max_positions": 8192, "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in order[:layers]]}
 
 

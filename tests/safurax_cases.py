@@ -83,8 +83,8 @@ S_C = model(130, 84, 1e-5, 1.0, [
 ])
 # S: softmaxes that are sharp (a large scale on large keys): a single key, far back or at a window's edge, decides
 #    a row's result.
-S_S = model(150, 64, 1e-5, 3.0, [
-    {**diff(2, 1, 32, 32, 1.5, 0.5, factor=4.0), "mlp": None},
+S_S = model(150, 64, 1e-5, 2.5, [
+    {**diff(2, 1, 32, 32, 1.5, 0.45, factor=3.0), "mlp": None},
     {**latent2(2, 16, 16, 16, 24, 90, 2.0), "mlp": None},
     {**latent(2, 24, 16, 40, 24, 1.5), "mlp": None},
     {**latent2(2, 16, 16, 16, 24, 40, 2.0, kv_from=1), "mlp": None},
